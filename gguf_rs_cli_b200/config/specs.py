@@ -38,6 +38,8 @@ class LayerSpec:
     # further parts that the block arrangement wires in by name (kinds of the registry of extra parts), for instance
     # an input of the layer's own that depends on the token alone
     extras: Dict[str, PartSpec] = field(default_factory=dict)
+    # constants of the arrangement itself, for instance the factor of x in a sum that is normed
+    block_params: Dict[str, Any] = field(default_factory=dict)
 
 
 @dataclass(frozen=True)

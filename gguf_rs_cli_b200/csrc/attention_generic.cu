@@ -13,7 +13,7 @@
 // multiplied by sigmoid(gate) entry by entry, or by one number per head; the softmax's denominator may count one
 // more key that has no value (a sink), of score 0 or of a learned score per head (not scaled).  Instead of a window
 // the keys may come in chunks of `chunk` positions counted from the sequence's start: a token sees the earlier tokens of
-// its own chunk only.
+// its own chunk only.  A distance bias takes slopes[head] * (i - j) off the scaled score of query i and key j.
 #include <math.h>
 
 #include "common.cuh"
@@ -31,7 +31,8 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
     int nh, int nkv, int hd, int hdv, int v_row, const int* __restrict__ seq_of, const int* __restrict__ pos,
     const int* __restrict__ table, int table_width, int ring_pages, const TC* __restrict__ kc,
     const TC* __restrict__ vc, int window, float scale, int head_pages, int keep_first, const void* __restrict__ gate,
-    int gate_dtype, long long ldg, int gate_per_head, int sink, const float* __restrict__ sink_values, int chunk) {
+    int gate_dtype, long long ldg, int gate_per_head, int sink, const float* __restrict__ sink_values, int chunk,
+    const float* __restrict__ slopes) {
     int t = blockIdx.x, h = blockIdx.y;
     int b = seq_of[t];
     size_t orow = size_t(t) * ldo + size_t(h) * hdv;
@@ -49,6 +50,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
     const bool vec8 = hd % 8 == 0 && (reinterpret_cast<uintptr_t>(kc) & 15) == 0;     // key rows start on 16 bytes
     int lo = gb_first_visible(p, window, chunk);
     int g = h / (nh / nkv);
+    const float slope = slopes ? slopes[h] : 0.f;
     const int* trow = table + size_t(b) * table_width;
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     constexpr int C = MAX_HD / 32;
@@ -118,6 +120,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
             for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], gb_to_float(kr[d]), dot);
             s = dot * scale;
         }
+        if (slopes) s -= slope * float(p - j);               // an unseen key's score stays -infinity
         float m_new = fmaxf(m, gb_warp_max(s));
         float alpha = (m == -INFINITY) ? 0.f : expf(m - m_new);
         float pj = valid ? expf(s - m_new) : 0.f;
@@ -193,7 +196,7 @@ GB_API int gb_attention_generic(const void* q, int q_dtype, long long ldq, void*
                                 const int* table, int table_width, int ring_pages, const void* kcache,
                                 const void* vcache, int cache_dtype, int window, float scale, int head_pages, int keep_first,
                                 const void* gate, int gate_dtype, long long ldg, int gate_per_head, int sink,
-                                const float* sink_values, int chunk, cudaStream_t stream) {
+                                const float* sink_values, int chunk, const float* slopes, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(q_dtype) && gb_is_dtype(out_dtype) && gb_is_dtype(cache_dtype), "gb_attention_generic: bad dtype");
     GB_REQUIRE(hd > 0 && hd <= AG_MAX_HD, "gb_attention_generic: head_dim %d is not in 1..%d", hd, AG_MAX_HD);
     GB_REQUIRE(hdv > 0 && hdv <= AG_MAX_HD && v_row >= hdv, "gb_attention_generic: value size %d (rows of %d) is not in 1..%d", hdv, v_row, AG_MAX_HD);
@@ -208,7 +211,7 @@ GB_API int gb_attention_generic(const void* q, int q_dtype, long long ldq, void*
 #define AG_LAUNCH(TC, MAX_HD)                                                                                     \
     attention_generic_kernel<TC, MAX_HD><<<grid, AG_WARPS * 32, 0, stream>>>(                                     \
         q, q_dtype, ldq, out, out_dtype, ldo, nh, nkv, hd, hdv, v_row, seq_of, pos, table, table_width, ring_pages, \
-        (const TC*)kcache, (const TC*)vcache, window, scale, head_pages, window > 0 ? keep_first : 0, gate, gate_dtype, ldg, gate_per_head, sink, sink_values, chunk)
+        (const TC*)kcache, (const TC*)vcache, window, scale, head_pages, window > 0 ? keep_first : 0, gate, gate_dtype, ldg, gate_per_head, sink, sink_values, chunk, slopes)
     const bool small = hd <= 256 && hdv <= 256, mid = hd <= AG_MID_HD && hdv <= AG_MID_HD;
     if (cache_dtype == GB_F32) {
         if (small) AG_LAUNCH(float, 256);

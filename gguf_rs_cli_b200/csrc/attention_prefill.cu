@@ -49,6 +49,7 @@ struct ApParams {
     int sink;                        // the softmax's denominator counts one more key of score 0 that has no value
     const float* sink_values;        // ... or of the score sink_values[head] (not scaled); null: 0
     int chunk;                       // > 0: in a window's place, a token sees the earlier tokens of its own chunk of that many positions
+    const float* slopes;             // [nh] or null: a score loses slopes[head] * (its distance), after the scale (EXACT only)
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -149,6 +150,11 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
     const int pq0 = r0 < rows ? start + q0 + r0 : -1, pq1 = r1 < rows ? start + q0 + r1 : -1;
     const int lo0 = gb_first_visible(pq0, p.window, p.chunk), lo1 = gb_first_visible(pq1, p.window, p.chunk);
 
+    // with a distance bias the scores are brought into the exponent's units (and biased) before the softmax
+    const bool biased = EXACT && p.slopes;
+    const float slope2 = biased ? p.slopes[h] * 1.4426950408889634f : 0.f;
+    const float sl2 = biased ? 1.f : p.scale_log2;
+
     float o[OT][4];
 #pragma unroll
     for (int i = 0; i < OT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -190,6 +196,11 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
         float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
+            if (biased) {
+                const float d0 = float(pq0 - key0 - 8 * j), d1 = float(pq1 - key0 - 8 * j);
+                s[j][0] = s[j][0] * p.scale_log2 - slope2 * d0; s[j][1] = s[j][1] * p.scale_log2 - slope2 * (d0 - 1.f);
+                s[j][2] = s[j][2] * p.scale_log2 - slope2 * d1; s[j][3] = s[j][3] * p.scale_log2 - slope2 * (d1 - 1.f);
+            }
             if (need_mask) {
                 int ka = key0 + 8 * j, kb2 = ka + 1;
                 if (ka > pq0 || (ka < lo0 && ka >= keep)) s[j][0] = -INFINITY;
@@ -205,15 +216,15 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-        const float a0 = mn0 == -INFINITY ? 1.f : exp2f((m0 - mn0) * p.scale_log2);
-        const float a1 = mn1 == -INFINITY ? 1.f : exp2f((m1 - mn1) * p.scale_log2);
-        const float ms0 = mn0 == -INFINITY ? 0.f : mn0 * p.scale_log2, ms1 = mn1 == -INFINITY ? 0.f : mn1 * p.scale_log2;
+        const float a0 = mn0 == -INFINITY ? 1.f : exp2f((m0 - mn0) * sl2);
+        const float a1 = mn1 == -INFINITY ? 1.f : exp2f((m1 - mn1) * sl2);
+        const float ms0 = mn0 == -INFINITY ? 0.f : mn0 * sl2, ms1 = mn1 == -INFINITY ? 0.f : mn1 * sl2;
         float sum0 = 0.f, sum1 = 0.f;
         unsigned pf[NT][2];
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-            float p0 = exp2f(s[j][0] * p.scale_log2 - ms0), p1 = exp2f(s[j][1] * p.scale_log2 - ms0);
-            float p2 = exp2f(s[j][2] * p.scale_log2 - ms1), p3 = exp2f(s[j][3] * p.scale_log2 - ms1);
+            float p0 = exp2f(s[j][0] * sl2 - ms0), p1 = exp2f(s[j][1] * sl2 - ms0);
+            float p2 = exp2f(s[j][2] * sl2 - ms1), p3 = exp2f(s[j][3] * sl2 - ms1);
             sum0 += p0 + p1;
             sum1 += p2 + p3;
             if (EXACT) {
@@ -275,8 +286,8 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     if (p.sink) {
         const float sv = p.sink_values ? p.sink_values[h] * 1.4426950408889634f : 0.f;
-        if (m0 != -INFINITY) l0 += exp2f(sv - m0 * p.scale_log2);
-        if (m1 != -INFINITY) l1 += exp2f(sv - m1 * p.scale_log2);
+        if (m0 != -INFINITY) l0 += exp2f(sv - m0 * sl2);
+        if (m1 != -INFINITY) l1 += exp2f(sv - m1 * sl2);
     }
     float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
     const bool entry_gate = p.gate && !p.gate_per_head;
@@ -336,12 +347,13 @@ GB_API int gb_attention_prefill(const void* q, long long ldq, void* out, long lo
                                 const int* table, int table_width, int ring_pages, const void* kcache,
                                 const void* vcache, int window, float scale, int exact, int head_pages, int keep_first,
                                 const void* gate, long long ldg, int gate_per_head, int sink, const float* sink_values, int chunk,
-                                cudaStream_t stream) {
+                                const float* slopes, cudaStream_t stream) {
     GB_REQUIRE(gb_attention_prefill_supported(hd, GB_BF16, GB_BF16), "gb_attention_prefill: head_dim %d is not 64 or 128", hd);
     GB_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0, "gb_attention_prefill: bad head counts %d / %d", nh, nkv);
     GB_REQUIRE(n_tiles <= 65535, "gb_attention_prefill: %d tiles of queries are too many for one launch", n_tiles);
     GB_REQUIRE(window >= 0 && ring_pages > 0 && table_width > 0 && head_pages >= 0, "gb_attention_prefill: bad cache geometry");
     GB_REQUIRE(keep_first >= 0, "gb_attention_prefill: a negative number of kept positions");
+    GB_REQUIRE(!slopes || exact, "gb_attention_prefill: a distance bias goes with 32-bit weights");
     GB_REQUIRE(!gate || gate_per_head || ((ldg % 2) == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0), "gb_attention_prefill: misaligned gate");
     GB_REQUIRE((ldq % 8) == 0 && (ldo % 2) == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(kcache) & 15) == 0 && (reinterpret_cast<uintptr_t>(vcache) & 15) == 0,
@@ -353,7 +365,7 @@ GB_API int gb_attention_prefill(const void* q, long long ldq, void* out, long lo
     p.ldq = ldq; p.ldo = ldo; p.nh = nh; p.nkv = nkv; p.table_width = table_width; p.ring_pages = ring_pages;
     p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
     p.head_pages = head_pages; p.keep_first = keep_first; p.gate = (const __nv_bfloat16*)gate; p.ldg = ldg;
-    p.gate_per_head = gate_per_head; p.sink = sink; p.sink_values = sink_values; p.chunk = chunk;
+    p.gate_per_head = gate_per_head; p.sink = sink; p.sink_values = sink_values; p.chunk = chunk; p.slopes = slopes;
     if (exact) return hd == 64 ? launch_ap<64, true>(p, n_tiles, stream) : launch_ap<128, true>(p, n_tiles, stream);
     return hd == 64 ? launch_ap<64, false>(p, n_tiles, stream) : launch_ap<128, false>(p, n_tiles, stream);
 }

@@ -83,44 +83,52 @@ GB_API int gb_qk_norm_kv_write(void* q, const void* k, const void* v, int dtype,
 // written to qa, head h's part starting at entry h * qa_stride + qa_off of the token's row (qa may be q
 // itself: the rotation is then done in place).
 // Rotation: the first rot_dims entries of the part, pair (2i, 2i+1) by position * inv_freq[i], or with `halves` pair
-// (i, i + rot_dims/2); the rest pass unchanged.
+// (i, i + rot_dims/2); the rest pass unchanged.  rot_gain multiplies sine and cosine.  dkv null: a layer that reads another
+// layer's rows; only the queries are rotated.
 __global__ void latent_prep_kernel(const void* __restrict__ q, long long ldq, const void* __restrict__ dkv,
                                    long long ldd, int dtype, int H, int D, int Rd, int C, int rot_dims,
                                    const float* __restrict__ inv_freq, const void* __restrict__ w, int w_dtype, float eps,
                                    void* qa, long long lda, int qa_stride, int qa_off, void* __restrict__ row_out,
                                    const int* __restrict__ seq_of,
                                    const int* __restrict__ pos, const int* __restrict__ table, int table_width,
-                                   int ring_pages, void* __restrict__ cache, int cache_dtype, int halves) {
+                                   int ring_pages, void* __restrict__ cache, int cache_dtype, int halves, float rot_gain) {
     __shared__ float red[32];
     const int t = blockIdx.x;
     const int b = seq_of[t];
     if (b < 0) return;
     const int p = pos[t];
     const size_t drow = size_t(t) * size_t(ldd);
-    float ss = 0.f;
-    for (int d = threadIdx.x; d < C; d += blockDim.x) {
-        const float x = gb_load(dkv, dtype, drow + d);
-        ss = fmaf(x, x, ss);
-    }
-    ss = gb_warp_sum(ss);
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-    __syncthreads();
-    float tot = 0.f;
-    for (int wv = 0; wv < (blockDim.x >> 5); ++wv) tot += red[wv];
-    const float f = 1.f / sqrtf(tot / float(C) + eps);
-    const size_t crow = gb_kv_offset(table + size_t(b) * table_width, ring_pages, p, 0, 1, C + Rd);
     const size_t rrow = size_t(t) * (C + Rd);
-    for (int d = threadIdx.x; d < C; d += blockDim.x) {
-        const float cv = gb_load(dkv, dtype, drow + d) * f * gb_load(w, w_dtype, d);
-        gb_store(cache, cache_dtype, crow + d, cv);
-        if (row_out) gb_store(row_out, dtype, rrow + d, cv);
+    size_t crow = 0;
+    if (dkv) {
+        float ss = 0.f;
+        for (int d = threadIdx.x; d < C; d += blockDim.x) {
+            const float x = gb_load(dkv, dtype, drow + d);
+            ss = fmaf(x, x, ss);
+        }
+        ss = gb_warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        float tot = 0.f;
+        for (int wv = 0; wv < (blockDim.x >> 5); ++wv) tot += red[wv];
+        const float f = 1.f / sqrtf(tot / float(C) + eps);
+        crow = gb_kv_offset(table + size_t(b) * table_width, ring_pages, p, 0, 1, C + Rd);
+        for (int d = threadIdx.x; d < C; d += blockDim.x) {
+            const float cv = gb_load(dkv, dtype, drow + d) * f * gb_load(w, w_dtype, d);
+            gb_store(cache, cache_dtype, crow + d, cv);
+            if (row_out) gb_store(row_out, dtype, rrow + d, cv);
+        }
     }
     // rotated parts: item 0 is the shared key part, items 1..H the heads' query parts
     const int half = rot_dims / 2, pairs = Rd / 2;          // Rd even: checked by the caller
-    for (int idx = threadIdx.x; idx < (H + 1) * pairs; idx += blockDim.x) {
+    for (int idx = threadIdx.x + (dkv ? 0 : pairs); idx < (H + 1) * pairs; idx += blockDim.x) {
         const int item = idx / pairs, i = idx - item * pairs;
         float sn = 0.f, cs = 1.f;
-        if (i < half) sincosf(float(p) * inv_freq[i], &sn, &cs);
+        if (i < half) {
+            sincosf(float(p) * inv_freq[i], &sn, &cs);
+            sn *= rot_gain;
+            cs *= rot_gain;
+        }
         // the pair that angle i turns: neighbours (2i, 2i+1), or with `halves` entries (i, i + half); pairs behind the
         // rotated entries pass unchanged either way
         const int d0 = halves && i < half ? i : 2 * i, d1 = halves && i < half ? i + half : 2 * i + 1;
@@ -153,15 +161,15 @@ GB_API int gb_latent_prep(const void* q, long long ldq, const void* dkv, long lo
                           int C, int rot_dims, const float* inv_freq, const void* w, int w_dtype, float eps, void* qa,
                           long long lda, int qa_stride, int qa_off, void* row_out, const int* seq_of, const int* pos,
                           const int* table, int table_width, int ring_pages, void* cache, int cache_dtype, int halves,
-                          cudaStream_t stream) {
+                          float rot_gain, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(dtype) && gb_is_dtype(w_dtype) && gb_is_dtype(cache_dtype), "gb_latent_prep: bad dtype");
     GB_REQUIRE(H > 0 && D >= 0 && C > 0 && Rd >= 0 && Rd % 2 == 0 && rot_dims >= 0 && rot_dims <= Rd && rot_dims % 2 == 0,
                "gb_latent_prep: bad sizes heads=%d dim=%d rot_dim=%d kv_rank=%d rotated=%d", H, D, Rd, C, rot_dims);
     GB_REQUIRE(rot_dims == 0 || inv_freq, "gb_latent_prep: no table of frequencies");
-    GB_REQUIRE(table && cache && ring_pages > 0 && table_width >= 1 && eps > 0.f, "gb_latent_prep: cache missing");
+    GB_REQUIRE(!dkv || (table && cache && w && ring_pages > 0 && table_width >= 1 && eps > 0.f), "gb_latent_prep: cache missing");
     if (T == 0) return 0;
     latent_prep_kernel<<<T, 128, 0, stream>>>(q, ldq, dkv, ldd, dtype, H, D, Rd, C, rot_dims, inv_freq, w, w_dtype, eps, qa, lda,
-                                              qa_stride, qa_off, row_out, seq_of, pos, table, table_width, ring_pages, cache, cache_dtype, halves);
+                                              qa_stride, qa_off, row_out, seq_of, pos, table, table_width, ring_pages, cache, cache_dtype, halves, rot_gain);
     GB_LAUNCH_OK("gb_latent_prep");
     return 0;
 }
@@ -210,13 +218,15 @@ GB_API int gb_pack_latent_heads(const void* kv, long long ldkv, const void* row,
 // out[t, h*os + o] = sum_i x[t, h*xs + i] * W[h, i, o] for o < O: every head has a matrix [I, O] of its own
 // (row-major, heads one after the other).  32-bit FMAs.  A block takes HM_TOKENS tokens, one head and 32
 // output columns; its four warps take a quarter of the inputs each (in ascending i) and the quarters are
-// added in warp order, so a token's result depends on neither the batch nor timing.
+// added in warp order, so a token's result depends on neither the batch nor timing.  A gate multiplies every result by
+// sigmoid(gate[t, h*O + o]).
 constexpr int HM_TOKENS = 8;
 
 template <typename TX, typename TW>
 __global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__ x, long long ldx, int xs,
                                                           const TW* __restrict__ W, int I, int O, void* __restrict__ out,
-                                                          int out_dtype, long long ldo, int os, int T) {
+                                                          int out_dtype, long long ldo, int os, int T,
+                                                          const void* __restrict__ gate, int gate_dtype, long long ldg) {
     extern __shared__ float xt[];                     // [HM_TOKENS][I], then [4][HM_TOKENS][32] partial sums
     float* part = xt + HM_TOKENS * I;
     const int t0 = blockIdx.x * HM_TOKENS, h = blockIdx.y;
@@ -246,8 +256,9 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__
     for (int idx = threadIdx.x; idx < HM_TOKENS * 32; idx += 128) {
         const int tt = idx >> 5, ol = idx & 31, oo = blockIdx.z * 32 + ol;
         if (tt < nt && oo < O) {
-            const float v = ((part[(0 * HM_TOKENS + tt) * 32 + ol] + part[(1 * HM_TOKENS + tt) * 32 + ol]) +
+            float v = ((part[(0 * HM_TOKENS + tt) * 32 + ol] + part[(1 * HM_TOKENS + tt) * 32 + ol]) +
                              part[(2 * HM_TOKENS + tt) * 32 + ol]) + part[(3 * HM_TOKENS + tt) * 32 + ol];
+            if (gate) v *= 1.f / (1.f + expf(-gb_load(gate, gate_dtype, size_t(t0 + tt) * ldg + size_t(h) * O + oo)));
             gb_store(out, out_dtype, size_t(t0 + tt) * ldo + size_t(h) * os + oo, v);
         }
     }
@@ -255,7 +266,9 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__
 
 // x: head h's I inputs start at column h*xs of a row (rows ldx apart); out: its O results start at column h*os.
 GB_API int gb_head_matmul(const void* x, int x_dtype, long long ldx, int xs, const void* W, int w_dtype, int H, int I, int O,
-                          void* out, int out_dtype, long long ldo, int os, int T, cudaStream_t stream) {
+                          void* out, int out_dtype, long long ldo, int os, int T, const void* gate, int gate_dtype,
+                          long long ldg, cudaStream_t stream) {
+    GB_REQUIRE(!gate || gb_is_dtype(gate_dtype), "gb_head_matmul: bad gate dtype");
     GB_REQUIRE(gb_is_dtype(x_dtype) && gb_is_dtype(w_dtype) && gb_is_dtype(out_dtype), "gb_head_matmul: bad dtype");
     GB_REQUIRE(H > 0 && H <= 65535 && I > 0 && O > 0 && xs >= I && os >= O, "gb_head_matmul: bad sizes heads=%d in=%d out=%d", H, I, O);
     const size_t smem = (size_t(HM_TOKENS) * I + 4 * HM_TOKENS * 32) * sizeof(float);
@@ -264,7 +277,7 @@ GB_API int gb_head_matmul(const void* x, int x_dtype, long long ldx, int xs, con
     dim3 grid((T + HM_TOKENS - 1) / HM_TOKENS, H, (O + 31) / 32);
     GB_REQUIRE(grid.z <= 65535, "gb_head_matmul: too many outputs per head (%d)", O);
 #define HM_LAUNCH(TX, TW)                                                                                             \
-    head_matmul_kernel<TX, TW><<<grid, 128, smem, stream>>>((const TX*)x, ldx, xs, (const TW*)W, I, O, out, out_dtype, ldo, os, T)
+    head_matmul_kernel<TX, TW><<<grid, 128, smem, stream>>>((const TX*)x, ldx, xs, (const TW*)W, I, O, out, out_dtype, ldo, os, T, gate, gate_dtype, ldg)
     if (x_dtype == GB_F32 && w_dtype == GB_F32) HM_LAUNCH(float, float);
     else if (x_dtype == GB_BF16 && w_dtype == GB_BF16) HM_LAUNCH(__nv_bfloat16, __nv_bfloat16);
     else if (x_dtype == GB_BF16 && w_dtype == GB_F32) HM_LAUNCH(__nv_bfloat16, float);
@@ -281,6 +294,7 @@ GB_API int gb_head_matmul(const void* x, int x_dtype, long long ldx, int xs, con
 //                                                                                  null: no norm at all)
 //   rot_p: the first rot_dims entries of a head in pairs, (i, i + rot_dims/2) or (2i, 2i+1), by the angle
 //          p * inv_freq[i]; the other entries pass; inv_freq null: no rotation
+//   q_h is also multiplied by temp(p) = 1 + coef * ln(floor((p + 1) / every) + 1) when coef is not 0
 //   v_g <- (1 - lambda) v_g + lambda v_first_g   when v_first is given (another layer's values of the same token);
 //   first_out, when given, receives the token's own values as they came (for the layers that mix them in).
 // A head lies in shared memory (32-bit) between the norm and the rotation.  Cache positions follow the page table
@@ -300,6 +314,8 @@ struct HeadPrepParams {
     float lambda;
     void* first_out;
     long long ld_out;
+    float temp_coef;
+    int temp_every;
     const int *seq_of, *pos, *table;
     int table_width, ring_pages, head_pages;
     void *kcache, *vcache;
@@ -318,6 +334,7 @@ __global__ void __launch_bounds__(128) head_prep_kv_write_kernel(const HeadPrepP
     const size_t row = size_t(t) * size_t(a.ld);
     const int* trow = a.table + size_t(b) * a.table_width;
     const int half = a.inv_freq ? a.rot_dims / 2 : 0;
+    const float temp = a.temp_coef != 0.f ? 1.f + a.temp_coef * logf(float((p + 1) / a.temp_every) + 1.f) : 1.f;
     const int items = a.k ? H + 2 * G : H;          // a layer that reads another layer's keys and values prepares its queries only
     for (int item = warp; item < items; item += warps) {
         if (item < H + G) {
@@ -335,6 +352,8 @@ __global__ void __launch_bounds__(128) head_prep_kv_write_kernel(const HeadPrepP
                 const float f = 1.f / sqrtf(gb_warp_sum(ss) / float(D) + a.eps);
                 for (int d = lane; d < D; d += 32) buf[d] = buf[d] * f * gb_load(w, a.w_dtype, d);
             }
+            if (is_q && a.temp_coef != 0.f)
+                for (int d = lane; d < D; d += 32) buf[d] *= temp;
             __syncwarp();
             void* dst = is_q ? a.q : a.kcache;
             const int dt = is_q ? a.dtype : a.cache_dtype;
@@ -368,9 +387,10 @@ __global__ void __launch_bounds__(128) head_prep_kv_write_kernel(const HeadPrepP
 GB_API int gb_head_prep_kv_write(void* q, const void* k, const void* v, int dtype, long long ld, int T, int H, int G, int D,
                                  int Dv, const void* wq, const void* wk, int w_dtype, float eps, const float* inv_freq,
                                  int rot_dims, int pairing, const void* v_first, long long ld_first, float lambda,
-                                 void* first_out, long long ld_out, const int* seq_of, const int* pos, const int* table,
-                                 int table_width, int ring_pages, int head_pages, void* kcache, void* vcache,
+                                 void* first_out, long long ld_out, float temp_coef, int temp_every, const int* seq_of, const int* pos,
+                                 const int* table, int table_width, int ring_pages, int head_pages, void* kcache, void* vcache,
                                  int cache_dtype, cudaStream_t stream) {
+    GB_REQUIRE(temp_coef == 0.f || temp_every > 0, "gb_head_prep_kv_write: the temperature's period must be positive, got %d", temp_every);
     GB_REQUIRE(gb_is_dtype(dtype) && gb_is_dtype(cache_dtype), "gb_head_prep_kv_write: bad dtype");
     GB_REQUIRE(H > 0 && G > 0 && D > 0 && Dv > 0 && D <= 4096, "gb_head_prep_kv_write: bad sizes heads=%d kv_heads=%d dim=%d vdim=%d", H, G, D, Dv);
     GB_REQUIRE((wq == nullptr) == (wk == nullptr) && (!wq || (gb_is_dtype(w_dtype) && eps > 0.f)), "gb_head_prep_kv_write: bad norm");
@@ -381,7 +401,7 @@ GB_API int gb_head_prep_kv_write(void* q, const void* k, const void* v, int dtyp
     HeadPrepParams a;
     a.q = q; a.k = k; a.v = v; a.ld = ld; a.dtype = dtype; a.H = H; a.G = G; a.D = D; a.Dv = Dv; a.wq = wq; a.wk = wk;
     a.w_dtype = w_dtype; a.eps = eps; a.inv_freq = inv_freq; a.rot_dims = rot_dims; a.pairing = pairing; a.v_first = v_first;
-    a.ld_first = ld_first; a.lambda = lambda; a.first_out = first_out; a.ld_out = ld_out; a.seq_of = seq_of; a.pos = pos;
+    a.ld_first = ld_first; a.lambda = lambda; a.first_out = first_out; a.ld_out = ld_out; a.temp_coef = temp_coef; a.temp_every = temp_every > 0 ? temp_every : 1; a.seq_of = seq_of; a.pos = pos;
     a.table = table; a.table_width = table_width; a.ring_pages = ring_pages; a.head_pages = head_pages; a.kcache = kcache;
     a.vcache = vcache; a.cache_dtype = cache_dtype;
     head_prep_kv_write_kernel<<<T, 128, size_t(4) * D * sizeof(float), stream>>>(a);

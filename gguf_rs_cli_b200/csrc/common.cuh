@@ -120,8 +120,10 @@ __device__ __forceinline__ float gb_gate_act(float z, int act) {
     return z / (1.f + expf(-z));
 }
 
-// A gated unit with clamped inputs: g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
-__device__ __forceinline__ float gb_act_glu_clamped(float g, float u, float limit) {
+// An expert's gated unit.  limit > 0: with clamped inputs, g <- min(g, limit), u <- clamp(u, -limit, limit),
+// g sigmoid(1.702 g) (u + 1).  limit 0: the plain unit g sigmoid(g) u.
+__device__ __forceinline__ float gb_act_glu(float g, float u, float limit) {
+    if (limit <= 0.f) return g / (1.f + expf(-g)) * u;
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);

@@ -149,7 +149,7 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const void* __restrict_
 }
 
 // ---------------------------------------------------------------- experts, token by token
-// y[t, r, f] = unit(Wg[e] h_t, Wu[e] h_t)_f with e = ids[t, r]; unit = gb_act_glu_clamped.  One block per (token,
+// y[t, r, f] = unit(Wg[e] h_t, Wu[e] h_t)_f with e = ids[t, r]; unit = gb_act_glu.  One block per (token,
 // choice) and slice of 32 features; the token's row lies in shared memory as 32-bit floats, a warp takes a feature at a
 // time and its lanes share the two matrix rows in pieces of eight (bfloat16) or four (float32) entries.
 // a lane's share of the product of a matrix row with the row in shared memory; the caller sums over the lanes
@@ -213,7 +213,7 @@ __global__ void __launch_bounds__(128) moe_gate_up_kernel(const void* __restrict
         float u = moe_row_dot<TW>(wu + row, moe_hs, K, lane);
         g = gb_warp_sum(g);
         u = gb_warp_sum(u);
-        if (lane == 0) gb_store(y, y_dtype, size_t(pair) * F + f, gb_act_glu_clamped(g, u, limit));
+        if (lane == 0) gb_store(y, y_dtype, size_t(pair) * F + f, gb_act_glu(g, u, limit));
     }
 }
 
@@ -282,7 +282,7 @@ GB_API int gb_moe_gate_up(const void* h, int h_dtype, long long ldh, int T, int 
                           const void* wg, const void* wu, int w_dtype, float limit, void* y, int y_dtype, int n_real,
                           cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(h_dtype) && gb_is_dtype(w_dtype) && gb_is_dtype(y_dtype), "gb_moe_gate_up: bad dtype");
-    GB_REQUIRE(K > 0 && F > 0 && top > 0 && limit > 0.f, "gb_moe_gate_up: bad sizes K=%d F=%d top=%d limit=%g", K, F, top, limit);
+    GB_REQUIRE(K > 0 && F > 0 && top > 0 && limit >= 0.f, "gb_moe_gate_up: bad sizes K=%d F=%d top=%d limit=%g", K, F, top, limit);
     if (T == 0) return 0;
     const size_t smem = size_t(K) * 4;
     dim3 grid(T * top, (F + MOE_SLICE - 1) / MOE_SLICE);
@@ -300,7 +300,7 @@ GB_API int gb_moe_gate_up(const void* h, int h_dtype, long long ldh, int T, int 
 }
 
 // y [T, top, F]; wd [E, N, F] contiguous; z float32 [T * top, N] scratch; out float32 [T, N] contiguous (added to when
-// accumulate).  Experts numbered n_real and above are identity experts: their pairs' rows are the tokens' own rows h
+// accumulate), or null: the pairs' rows stay in z for a caller that sums them itself.  Experts numbered n_real and above are identity experts: their pairs' rows are the tokens' own rows h
 // [T, N] (rows ldh apart).  Two launches.
 GB_API int gb_moe_down(const void* y, int y_dtype, int T, int F, int N, int top, const int* ids, const float* weights,
                        const void* wd, int w_dtype, float* z, float* out, int accumulate, int n_real, const void* h, int h_dtype,
@@ -320,6 +320,7 @@ GB_API int gb_moe_down(const void* y, int y_dtype, int T, int F, int N, int top,
         moe_down_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>(y, y_dtype, F, N, ids, (const __nv_bfloat16*)wd, z, h ? n_real : 0x7fffffff, h, h_dtype, ldh, top);
     }
     GB_LAUNCH_OK("gb_moe_down");
+    if (!out) return 0;
     const long long total = (long long)T * N;
     moe_pair_sum_kernel<<<unsigned((total + 255) / 256), 256, 0, stream>>>(z, weights, top, N, out, accumulate, total);
     GB_LAUNCH_OK("gb_moe_down (sum)");
@@ -327,6 +328,22 @@ GB_API int gb_moe_down(const void* y, int y_dtype, int T, int F, int N, int top,
 }
 
 // ---------------------------------------------------------------- activations of whole buffers
+// bfloat16, eight entries per thread
+__global__ void __launch_bounds__(256) unary_act_vec_kernel(uint4* __restrict__ x, long long n8, int act) {
+    const long long i = blockIdx.x * 256LL + threadIdx.x;
+    gb_grid_launch_dependents();
+    gb_grid_wait();
+    if (i >= n8) return;
+    uint4 v = x[i];
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(p[e]);
+        p[e] = __floats2bfloat162_rn(gb_act_unary(f.x, act), gb_act_unary(f.y, act));
+    }
+    x[i] = v;
+}
+
 __global__ void unary_act_kernel(void* __restrict__ x, int dtype, long long n, int act) {
     const long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x;
     if (i < n) gb_store(x, dtype, size_t(i), gb_act_unary(gb_load(x, dtype, size_t(i)), act));
@@ -354,6 +371,11 @@ GB_API int gb_unary_act_rows(void* x, int dtype, int rows, int cols, long long l
 GB_API int gb_unary_act(void* x, int dtype, long long n, int act, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(dtype) && act >= 1 && act <= 4, "gb_unary_act: bad dtype or activation %d", act);
     if (n == 0) return 0;
+    if (dtype == GB_BF16 && n % 8 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+        gb_launch(unary_act_vec_kernel, dim3(unsigned((n / 8 + 255) / 256)), dim3(256), 0, stream, (uint4*)x, n / 8, act);
+        GB_LAUNCH_OK("gb_unary_act");
+        return 0;
+    }
     unary_act_kernel<<<unsigned((n + 255) / 256), 256, 0, stream>>>(x, dtype, n, act);
     GB_LAUNCH_OK("gb_unary_act");
     return 0;
@@ -365,12 +387,12 @@ __global__ void glu_clamped_kernel(const void* __restrict__ gu, long long ld, vo
     if (i >= (long long)T * F) return;
     const long long t = i / F;
     const int f = int(i - t * F);
-    gb_store(out, dtype, size_t(i), gb_act_glu_clamped(gb_load(gu, dtype, size_t(t) * ld + f), gb_load(gu, dtype, size_t(t) * ld + F + f), limit));
+    gb_store(out, dtype, size_t(i), gb_act_glu(gb_load(gu, dtype, size_t(t) * ld + f), gb_load(gu, dtype, size_t(t) * ld + F + f), limit));
 }
 
-// gate_up [T, 2F] (gate in the first F columns, rows ld apart) -> out [T, F] contiguous = gb_act_glu_clamped(gate, up).
+// gate_up [T, 2F] (gate in the first F columns, rows ld apart) -> out [T, F] contiguous = gb_act_glu(gate, up).
 GB_API int gb_glu_clamped(const void* gate_up, long long ld, void* out, int T, int F, int dtype, float limit, cudaStream_t stream) {
-    GB_REQUIRE(gb_is_dtype(dtype) && F > 0 && limit > 0.f, "gb_glu_clamped: bad arguments");
+    GB_REQUIRE(gb_is_dtype(dtype) && F > 0 && limit >= 0.f, "gb_glu_clamped: bad arguments");
     if (T == 0) return 0;
     const long long n = (long long)T * F;
     glu_clamped_kernel<<<unsigned((n + 255) / 256), 256, 0, stream>>>(gate_up, ld, out, T, F, dtype, limit);

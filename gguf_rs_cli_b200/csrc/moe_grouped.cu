@@ -220,12 +220,12 @@ __global__ void __launch_bounds__(MG_THREADS, 5) moe_grouped_kernel(const MgPara
         if (GLU) {
             __nv_bfloat16* y = reinterpret_cast<__nv_bfloat16*>(p.out);
             if (pair0 >= 0) {
-                y[size_t(pair0) * p.N + n] = __float2bfloat16_rn(gb_act_glu_clamped(acc[0][mi][j][0], acc[NB - 1][mi][j][0], p.limit));
-                if (two) y[size_t(pair0) * p.N + n + 1] = __float2bfloat16_rn(gb_act_glu_clamped(acc[0][mi][j][1], acc[NB - 1][mi][j][1], p.limit));
+                y[size_t(pair0) * p.N + n] = __float2bfloat16_rn(gb_act_glu(acc[0][mi][j][0], acc[NB - 1][mi][j][0], p.limit));
+                if (two) y[size_t(pair0) * p.N + n + 1] = __float2bfloat16_rn(gb_act_glu(acc[0][mi][j][1], acc[NB - 1][mi][j][1], p.limit));
             }
             if (pair1 >= 0) {
-                y[size_t(pair1) * p.N + n] = __float2bfloat16_rn(gb_act_glu_clamped(acc[0][mi][j][2], acc[NB - 1][mi][j][2], p.limit));
-                if (two) y[size_t(pair1) * p.N + n + 1] = __float2bfloat16_rn(gb_act_glu_clamped(acc[0][mi][j][3], acc[NB - 1][mi][j][3], p.limit));
+                y[size_t(pair1) * p.N + n] = __float2bfloat16_rn(gb_act_glu(acc[0][mi][j][2], acc[NB - 1][mi][j][2], p.limit));
+                if (two) y[size_t(pair1) * p.N + n + 1] = __float2bfloat16_rn(gb_act_glu(acc[0][mi][j][3], acc[NB - 1][mi][j][3], p.limit));
             }
         } else {
             float* z = reinterpret_cast<float*>(p.out);
@@ -266,14 +266,15 @@ GB_API long long gb_moe_grouped_scratch_ints(int T, int top, int E) {
 }
 
 // h bfloat16 [T, K] rows ldh apart; ids [T, top], weights [T, top]; wg, wu [E, F, K], wd [E, N, F] bfloat16 contiguous;
-// y bfloat16 [T*top, F], z float [T*top, N] scratch; out float [T, N] (added to when accumulate).  E counts all experts
+// y bfloat16 [T*top, F], z float [T*top, N] scratch; out float [T, N] (added to when accumulate; null: the pairs' rows stay
+// in z).  E counts all experts
 // that ids may name; those numbered n_real and above are identity experts without matrices (then N = K).
 GB_API int gb_moe_grouped(const void* h, long long ldh, int T, int K, int F, int N, int E, int top, const int* ids,
                           const float* weights, const void* wg, const void* wu, const void* wd, float limit, void* y, float* z,
                           int* scratch, float* out, int accumulate, int n_real, cudaStream_t stream) {
     GB_REQUIRE(n_real > 0 && n_real <= E && (n_real == E || N == K), "gb_moe_grouped: %d of %d experts have matrices (rows of %d and %d)", n_real, E, K, N);
     GB_REQUIRE(gb_moe_grouped_supported(K, F), "gb_moe_grouped: sizes K=%d F=%d must be multiples of 8", K, F);
-    GB_REQUIRE(E > 0 && E <= 1024 && top > 0 && N > 0 && limit > 0.f && (ldh % 8) == 0, "gb_moe_grouped: bad sizes");
+    GB_REQUIRE(E > 0 && E <= 1024 && top > 0 && N > 0 && limit >= 0.f && (ldh % 8) == 0, "gb_moe_grouped: bad sizes");
     GB_REQUIRE(((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(wg) | reinterpret_cast<uintptr_t>(wu) |
                  reinterpret_cast<uintptr_t>(wd) | reinterpret_cast<uintptr_t>(y)) & 15) == 0, "gb_moe_grouped: misaligned operands");
     if (T == 0) return 0;
@@ -303,6 +304,7 @@ GB_API int gb_moe_grouped(const void* h, long long ldh, int T, int K, int F, int
     p.N = N; p.K = F;
     moe_grouped_kernel<false><<<dim3((N + MG_BN - 1) / MG_BN, max_tiles), MG_THREADS, SMEM_ONE, stream>>>(p);
     GB_LAUNCH_OK("gb_moe_grouped (down)");
+    if (!out) return 0;
     const long long total = (long long)T * N;
     MoeIdentity id;
     id.ids = n_real < E ? ids : nullptr; id.h = h; id.ldh = ldh; id.n_real = n_real; id.h_dtype = GB_BF16;

@@ -80,15 +80,17 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
                       kcache: torch.Tensor, vcache: Optional[torch.Tensor], window: int, scale: float,
                       v_dim: Optional[int] = None, keep_first: int = 0, head_pages: int = 0,
                       gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                      chunk: int = 0) -> torch.Tensor:
+                      chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """v_dim: entries of a value when they differ from a key's head_dim.  vcache None: the values are the
     first v_dim entries of the key rows themselves (one latent row per position serves as key and value).
     keep_first: with a window, the sequence's first positions that stay visible behind it; their pages are the first
     head_pages entries of the page table, in front of the ring.  gate [T, heads*v_dim]: the result is multiplied by
     sigmoid(gate); a gate [T, heads] holds one number per head.  sink: the softmax's denominator counts one more key
     of score 0 that has no value, or of the score sink_values[head] (float32 [heads], not scaled).  chunk: instead of a
-    window, a token sees the earlier tokens of its own chunk of that many positions, counted from the sequence's start."""
+    window, a token sees the earlier tokens of its own chunk of that many positions, counted from the sequence's start.
+    slopes float32 [heads]: slopes[head] times the distance of query and key is taken off every scaled score."""
     _cuda(q, out, seq_of, pos, table, kcache, vcache, gate, sink_values)
+    _check_slopes(slopes, n_heads)
     T = q.shape[0]
     per_head = _gate_per_head(gate, out, n_heads)
     assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == n_heads and sink_values.is_contiguous())
@@ -101,8 +103,12 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
          ptr(kcache), ptr(kcache if vcache is None else vcache), dtype_code(kcache), int(window or 0), float(scale),
          int(head_pages), int(keep_first or 0), ptr(gate), 0 if gate is None else dtype_code(gate),
          0 if gate is None else gate.stride(0), int(per_head), int(bool(sink) or sink_values is not None), ptr(sink_values),
-         int(chunk or 0), stream_ptr())
+         int(chunk or 0), ptr(slopes), stream_ptr())
     return out
+
+
+def _check_slopes(slopes: Optional[torch.Tensor], n_heads: int) -> None:
+    assert slopes is None or (slopes.is_cuda and slopes.dtype == torch.float32 and slopes.numel() == n_heads and slopes.is_contiguous())
 
 
 def _gate_per_head(gate: Optional[torch.Tensor], out: torch.Tensor, n_heads: int) -> bool:
@@ -396,11 +402,13 @@ def head_prep_kv_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
                        q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                        inv_freq: Optional[torch.Tensor], rotary_dim: int, pairing: int, v_first: Optional[torch.Tensor],
                        mix: float, first_out: Optional[torch.Tensor], seq_of: torch.Tensor, pos: torch.Tensor,
-                       table: torch.Tensor, ring_pages: int, head_pages: int, kcache: torch.Tensor, vcache: torch.Tensor) -> None:
+                       table: torch.Tensor, ring_pages: int, head_pages: int, kcache: torch.Tensor, vcache: torch.Tensor,
+                       temp_coef: float = 0.0, temp_every: int = 1) -> None:
     """q, k, v: column slices of one row-major buffer.  Per head: RMS norm with a weight of `dim` entries that all
     heads share (q_weight, k_weight; None: no norm), then the rotation of the first rotary_dim entries (inv_freq None:
     none); q in place, k into the cache.  v <- (1 - mix) v + mix v_first when v_first [T, kv_heads*vdim] is given,
-    into the cache; first_out receives v as it came."""
+    into the cache; first_out receives v as it came.  v may be k itself: the keys as projected are then the values.
+    temp_coef: q is also multiplied by 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)."""
     _cuda(q, k, v, q_weight, k_weight, inv_freq, v_first, first_out, seq_of, pos, table, kcache, vcache)
     T, ld = q.shape[0], q.stride(0)
     if k is None:                       # a layer that reads another layer's keys and values: its queries only
@@ -415,8 +423,8 @@ def head_prep_kv_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
     call("gb_head_prep_kv_write", ptr(q), ptr(k), ptr(v), dtype_code(q), ld, T, n_heads, n_kv_heads, dim, vdim, ptr(q_weight),
          ptr(k_weight), 0 if q_weight is None else dtype_code(q_weight), float(eps), ptr(inv_freq), int(rotary_dim), int(pairing),
          ptr(v_first), 0 if v_first is None else v_first.stride(0), float(mix), ptr(first_out),
-         0 if first_out is None else first_out.stride(0), ptr(seq_of), ptr(pos), ptr(table), table.shape[1], int(ring_pages),
-         int(head_pages), ptr(kcache), ptr(vcache), 0 if kcache is None else dtype_code(kcache), stream_ptr())
+         0 if first_out is None else first_out.stride(0), float(temp_coef), int(temp_every), ptr(seq_of), ptr(pos), ptr(table),
+         table.shape[1], int(ring_pages), int(head_pages), ptr(kcache), ptr(vcache), 0 if kcache is None else dtype_code(kcache), stream_ptr())
 
 
 def moe_route(logits: torch.Tensor, n_groups: int, keep: int, top: int, scale: float, ids: torch.Tensor,
@@ -455,7 +463,7 @@ def moe_router(x: torch.Tensor, w: torch.Tensor, n_groups: int, keep: int, top: 
 def moe_gate_up(h: torch.Tensor, ids: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor, limit: float,
                 y: torch.Tensor, identity: int = 0) -> torch.Tensor:
     """y[t, r, :] = unit(W_gate[e] h_t, W_up[e] h_t), e = ids[t, r]; unit(g, u) = g' sigmoid(1.702 g') (u' + 1) with
-    g' = min(g, limit), u' = clamp(u, -limit, limit).  w_gate, w_up [experts, F, K]; token by token on the CUDA cores."""
+    g' = min(g, limit), u' = clamp(u, -limit, limit); with limit 0 the plain unit g sigmoid(g) u.  w_gate, w_up [experts, F, K]; token by token on the CUDA cores."""
     _cuda(h, ids, w_gate, w_up, y)
     T, K = h.shape
     E, F, _ = w_gate.shape
@@ -467,15 +475,17 @@ def moe_gate_up(h: torch.Tensor, ids: torch.Tensor, w_gate: torch.Tensor, w_up: 
     return y
 
 
-def moe_down(y: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_down: torch.Tensor, out: torch.Tensor,
+def moe_down(y: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_down: torch.Tensor, out: Optional[torch.Tensor],
              accumulate: bool = False, ws=None, identity: int = 0, h: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] (+)= sum_r weights[t, r] W_down[ids[t, r]] y[t, r]; w_down [experts, N, F]; out float32 [T, N].  Every pair's
-    row first (32-bit, in a buffer of the workspace `ws` when given), then the weighted sum per token: two launches."""
+    row first (32-bit, in a buffer of the workspace `ws` when given), then the weighted sum per token: two launches.
+    out None: one launch; the pairs' rows [T*top, N] are returned unsummed."""
     _cuda(y, ids, weights, w_down, out)
     T, top, F = y.shape
     E, N, _ = w_down.shape
-    assert y.is_contiguous() and w_down.is_contiguous() and w_down.shape == (E, N, F) and out.shape == (T, N)
-    assert out.dtype == torch.float32 and out.is_contiguous() and ids.shape == (T, top) and weights.shape == (T, top)
+    assert y.is_contiguous() and w_down.is_contiguous() and w_down.shape == (E, N, F)
+    assert out is None or (out.shape == (T, N) and out.dtype == torch.float32 and out.is_contiguous())
+    assert ids.shape == (T, top) and weights.shape == (T, top) and (out is not None or not identity)
     z = ws.get("moe.rows", (T * top, N), torch.float32) if ws is not None else torch.empty(T * top, N, dtype=torch.float32, device=y.device)
     # identity experts (ids from the number of matrices on, `identity` of them) give the token's own row h [T, N]
     assert not identity or (h is not None and h.shape == (T, N) and h.stride(1) == 1)
@@ -483,6 +493,9 @@ def moe_down(y: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_down: 
     call("gb_moe_down", ptr(y), dtype_code(y), T, F, N, top, ptr(ids), ptr(weights), ptr(w_down), dtype_code(w_down), ptr(z),
          ptr(out), int(bool(accumulate)), E, ptr(own), 0 if own is None else dtype_code(own), 0 if own is None else own.stride(0),
          stream_ptr())
+    if out is None:
+        native.count_launches(-1)
+        return z
     return out
 
 
@@ -493,16 +506,18 @@ def moe_grouped_supported(h: torch.Tensor, w_gate: torch.Tensor) -> bool:
 
 
 def moe_grouped(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor,
-                w_down: torch.Tensor, limit: float, out: torch.Tensor, ctx, accumulate: bool = False, identity: int = 0) -> torch.Tensor:
+                w_down: torch.Tensor, limit: float, out: Optional[torch.Tensor], ctx, accumulate: bool = False, identity: int = 0) -> torch.Tensor:
     """The routed experts of a step of many tokens on the tensor cores: the (token, choice) pairs sorted by expert on
     the device, gate and up with the clamped unit, down, and the weighted sum per token; what moe_gate_up and moe_down
-    give, up to the rounding of bfloat16 unit outputs.  Four launches."""
+    give, up to the rounding of bfloat16 unit outputs.  Four launches; with out None three, and the pairs' rows [T*top, N]
+    are returned unsummed."""
     _cuda(h, ids, weights, w_gate, w_up, w_down, out)
     T, K = h.shape
     E, F, _ = w_gate.shape
     N, top = w_down.shape[1], ids.shape[1]
-    assert w_gate.shape == w_up.shape == (E, F, K) and w_down.shape == (E, N, F) and out.shape == (T, N) and out.dtype == torch.float32
-    assert w_gate.is_contiguous() and w_up.is_contiguous() and w_down.is_contiguous() and out.is_contiguous()
+    assert w_gate.shape == w_up.shape == (E, F, K) and w_down.shape == (E, N, F) and (out is not None or not identity)
+    assert out is None or (out.shape == (T, N) and out.dtype == torch.float32 and out.is_contiguous())
+    assert w_gate.is_contiguous() and w_up.is_contiguous() and w_down.is_contiguous()
     assert ids.shape == weights.shape == (T, top) and ids.is_contiguous() and weights.is_contiguous()
     y = ctx.ws.get("moe.units", (T, top, F), torch.bfloat16)
     z = ctx.ws.get("moe.rows", (T * top, N), torch.float32)
@@ -510,21 +525,26 @@ def moe_grouped(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     scratch = ctx.ws.get("moe.sorted", (native.library().gb_moe_grouped_scratch_ints(T, top, n_all),), torch.int32)
     call("gb_moe_grouped", ptr(h), h.stride(0), T, K, F, N, n_all, top, ptr(ids), ptr(weights), ptr(w_gate), ptr(w_up), ptr(w_down),
          float(limit), ptr(y), ptr(z), ptr(scratch), ptr(out), int(bool(accumulate)), E, stream_ptr())
+    if out is None:
+        native.count_launches(-1)
+        return z
     return out
 
 
 def moe_by_expert(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor,
-                  w_down: torch.Tensor, limit: float, out: torch.Tensor, ctx, accumulate: bool = False, identity: int = 0) -> torch.Tensor:
+                  w_down: torch.Tensor, limit: float, out: Optional[torch.Tensor], ctx, accumulate: bool = False, identity: int = 0):
     """The routed experts of a step of very many tokens as ordinary products, expert by expert, on the tcgen05 product
     kernels: the pairs sorted by expert and the tokens' rows gathered in that order on the device; the experts' offsets
     read on the host (one wait per call: such steps are prompts, which no graph captures); per expert gate, up and down
-    over its own rows; the clamped unit over all rows at once; the weighted sum per token in choice order."""
+    over its own rows; the clamped unit over all rows at once; the weighted sum per token in choice order.  out None: no sum;
+    returns the rows [T*top, N] in the experts' order and place_of [T*top], where each pair's row lies."""
     _cuda(h, ids, weights, w_gate, w_up, w_down, out)
     T, K = h.shape
     E, F, _ = w_gate.shape
     N, top = w_down.shape[1], ids.shape[1]
     P = T * top
-    assert h.dtype == torch.bfloat16 and w_gate.dtype == torch.bfloat16 and out.dtype == torch.float32 and out.shape == (T, N)
+    assert h.dtype == torch.bfloat16 and w_gate.dtype == torch.bfloat16 and (out is not None or not identity)
+    assert out is None or (out.dtype == torch.float32 and out.shape == (T, N))
     lib = native.library()
     n_all = E + int(identity)                 # identity experts are sorted behind the others; their rows are never multiplied
     scratch = ctx.ws.get("moe.sorted", (lib.gb_moe_grouped_scratch_ints(T, top, n_all),), torch.int32)
@@ -546,6 +566,8 @@ def moe_by_expert(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_g
         a, b = at[e], at[e + 1]
         if b > a:
             gemm(y[a:b], w_down[e], None, z[a:b])
+    if out is None:
+        return z, place_of
     call("gb_moe_combine_sorted", ptr(z), ptr(place_of), ptr(weights), T, top, N, ptr(out), int(bool(accumulate)),
          ptr(ids) if identity else None, E, ptr(h), dtype_code(h), h.stride(0), stream_ptr())
     return out
@@ -568,7 +590,7 @@ def unary_act_(x: torch.Tensor, activation: str) -> torch.Tensor:
 
 def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float) -> torch.Tensor:
     """gate_up [T, 2F], gate in the first F columns; out[t, i] = g' sigmoid(1.702 g') (u' + 1) with the inputs clamped
-    as in moe_gate_up."""
+    as in moe_gate_up (limit 0: the plain unit)."""
     _cuda(gate_up, out)
     T, F = out.shape
     assert gate_up.shape == (T, 2 * F) and gate_up.stride(1) == 1 and out.is_contiguous() and out.dtype == gate_up.dtype
@@ -593,29 +615,32 @@ def qk_norm_kv_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[tor
          0 if kcache is None else dtype_code(kcache), stream_ptr())
 
 
-def latent_prep(q: torch.Tensor, dkv: torch.Tensor, n_heads: int, dim: int, rot_dim: int, kv_rank: int, rot_dims: int,
-                inv_freq: Optional[torch.Tensor], weight: torch.Tensor, eps: float, qa: Optional[torch.Tensor],
+def latent_prep(q: torch.Tensor, dkv: Optional[torch.Tensor], n_heads: int, dim: int, rot_dim: int, kv_rank: int, rot_dims: int,
+                inv_freq: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, qa: Optional[torch.Tensor],
                 seq_of: torch.Tensor, pos: torch.Tensor, table: torch.Tensor, ring_pages: int, cache: torch.Tensor,
-                row_out: Optional[torch.Tensor] = None, halves: bool = False) -> None:
+                row_out: Optional[torch.Tensor] = None, halves: bool = False, gain: float = 1.0) -> None:
     """Latent attention in front of the attention kernel: dkv [T, kv_rank + rot_dim] gives the cache row
     (RMS-normed latent, rotated shared key part; also copied to row_out [T, kv_rank + rot_dim] when given); the
     heads' rotated query parts go to qa [T, heads*(kv_rank + rot_dim)] behind the kv_rank entries that
-    head_matmul fills, or, with qa None, are rotated in place in q."""
+    head_matmul fills, or, with qa None, are rotated in place in q.  gain multiplies sine and cosine.  dkv None: a layer that
+    reads another layer's rows; only the queries are rotated."""
     _cuda(q, dkv, inv_freq, weight, qa, seq_of, pos, table, cache, row_out)
     T = q.shape[0]
-    assert q.stride(1) == 1 and dkv.stride(1) == 1 and q.dtype == dkv.dtype
-    assert q.shape[1] == n_heads * (dim + rot_dim) and dkv.shape[1] == kv_rank + rot_dim
-    assert cache.shape[-1] == kv_rank + rot_dim and weight.numel() == kv_rank
+    assert q.stride(1) == 1 and q.shape[1] == n_heads * (dim + rot_dim) and cache.shape[-1] == kv_rank + rot_dim
+    if dkv is not None:
+        assert dkv.stride(1) == 1 and q.dtype == dkv.dtype and dkv.shape[1] == kv_rank + rot_dim and weight.numel() == kv_rank
+    else:
+        assert row_out is None
     if qa is None:
         qa, stride, off = q, dim + rot_dim, dim
     else:
         stride, off = kv_rank + rot_dim, kv_rank
         assert qa.shape == (T, n_heads * (kv_rank + rot_dim)) and qa.stride(1) == 1 and qa.dtype == q.dtype
     assert row_out is None or (row_out.shape == (T, kv_rank + rot_dim) and row_out.is_contiguous() and row_out.dtype == q.dtype)
-    call("gb_latent_prep", ptr(q), q.stride(0), ptr(dkv), dkv.stride(0), dtype_code(q), T, n_heads, dim, rot_dim, kv_rank,
-         rot_dims, ptr(inv_freq), ptr(weight), dtype_code(weight), float(eps), ptr(qa), qa.stride(0), stride, off,
+    call("gb_latent_prep", ptr(q), q.stride(0), ptr(dkv), 0 if dkv is None else dkv.stride(0), dtype_code(q), T, n_heads, dim, rot_dim, kv_rank,
+         rot_dims, ptr(inv_freq), ptr(weight), 0 if weight is None else dtype_code(weight), float(eps), ptr(qa), qa.stride(0), stride, off,
          ptr(row_out), ptr(seq_of), ptr(pos), ptr(table), table.shape[1], ring_pages, ptr(cache), dtype_code(cache),
-         int(bool(halves)), stream_ptr())
+         int(bool(halves)), float(gain), stream_ptr())
 
 
 def pack_latent_heads(kv: torch.Tensor, row: torch.Tensor, n_heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int,
@@ -668,15 +693,19 @@ def latent_decode(qa: torch.Tensor, out: torch.Tensor, n_heads: int, kv_rank: in
     return out
 
 
-def head_matmul(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int) -> torch.Tensor:
-    """out[t, h*out_head_stride + o] = sum_i x[t, h*x_head_stride + i] * w[h, i, o]; w [heads, in, out]."""
-    _cuda(x, w, out)
+def head_matmul(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
+                gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t, h*out_head_stride + o] = sum_i x[t, h*x_head_stride + i] * w[h, i, o]; w [heads, in, out].  gate [T, heads*out]:
+    every result is multiplied by its sigmoid."""
+    _cuda(x, w, out, gate)
     H, I, O = w.shape
     T = x.shape[0]
     assert w.is_contiguous() and x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == T
     assert x.shape[1] >= (H - 1) * x_head_stride + I and out.shape[1] >= (H - 1) * out_head_stride + O
+    assert gate is None or (gate.shape == (T, H * O) and gate.stride(1) == 1)
     call("gb_head_matmul", ptr(x), dtype_code(x), x.stride(0), int(x_head_stride), ptr(w), dtype_code(w), H, I, O, ptr(out),
-         dtype_code(out), out.stride(0), int(out_head_stride), T, stream_ptr())
+         dtype_code(out), out.stride(0), int(out_head_stride), T, ptr(gate), 0 if gate is None else dtype_code(gate),
+         0 if gate is None else gate.stride(0), stream_ptr())
     return out
 
 
@@ -731,6 +760,43 @@ def norm_sandwich(x: Optional[torch.Tensor], y: Optional[torch.Tensor], weight: 
          0 if y2 is None else dtype_code(y2), 0 if y2 is None else y2.stride(0), ptr(wy), ptr(wy2), float(mix), ptr(weight),
          ptr(next_weight), dtype_code(ws[0]), float(eps), ptr(h), 0 if h is None else dtype_code(h), ptr(xb), ptr(u_out), T, E,
          stream_ptr())
+
+
+def layernorm(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, eps: float, alpha: float = 1.0,
+              routed: Optional[tuple] = None, rows: Optional[torch.Tensor] = None, h: Optional[torch.Tensor] = None,
+              xb: Optional[torch.Tensor] = None, write_x: bool = True) -> None:
+    """LN(v) = (v - mean v) / sqrt(mean((v - mean v)^2) + eps) * weight of v = alpha x + y + the routed rows, row by row in
+    32-bit: into x (float32 [T, E]; write_x), its bfloat16 copy xb and h (each when given).  routed = (z, weights,
+    place_of): rows z float32 [T*top, E] of which token t takes sum_r weights[t, r] z[place_of[t*top + r]] (place_of None:
+    the pairs' own order).  rows: int32 row numbers to gather (then h has len(rows) rows)."""
+    z, wts, place = routed if routed is not None else (None, None, None)
+    _cuda(x, y, weight, z, wts, place, rows, h, xb)
+    T, E = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and weight.numel() == E and weight.is_contiguous()
+    assert y is None or (y.shape == (T, E) and y.stride(1) == 1)
+    top = 0
+    if z is not None:
+        top = wts.shape[1]
+        assert z.dtype == torch.float32 and z.shape == (T * top, E) and z.is_contiguous()
+        assert wts.dtype == torch.float32 and wts.shape == (T, top) and wts.is_contiguous()
+        assert place is None or (place.dtype == torch.int32 and place.numel() == T * top and place.is_contiguous())
+    n = T if rows is None else rows.numel()
+    assert h is None or (h.shape == (n, E) and h.is_contiguous())
+    assert rows is None or not (write_x or xb is not None)
+    assert xb is None or (xb.dtype == torch.bfloat16 and xb.shape == (T, E) and xb.is_contiguous())
+    call("gb_layernorm", ptr(x), ptr(y), 0 if y is None else dtype_code(y), 0 if y is None else y.stride(0), ptr(z), ptr(wts),
+         ptr(place), top, float(alpha), ptr(weight), dtype_code(weight), float(eps), ptr(rows), n, E, ptr(h),
+         0 if h is None else dtype_code(h), ptr(xb), int(write_x), stream_ptr())
+
+
+def rms_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """out[t,:] = x[t,:] / sqrt(mean(x[t,:]^2) + eps) * weight (32-bit sums); x may be a block of columns."""
+    _cuda(x, weight, out)
+    T, C = x.shape
+    assert x.stride(1) == 1 and out.stride(1) == 1 and out.shape == (T, C) and weight.numel() == C and weight.is_contiguous()
+    call("gb_rms_rows", ptr(x), dtype_code(x), x.stride(0), T, C, ptr(weight), dtype_code(weight), float(eps), ptr(out),
+         dtype_code(out), out.stride(0), stream_ptr())
+    return out
 
 
 def token_side_gate(a: torch.Tensor, table: torch.Tensor, offset: int, tokens: torch.Tensor, out: torch.Tensor,
@@ -959,18 +1025,19 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_head
                      splits: Optional[int] = None, mma: Optional[bool] = None, max_kv: Optional[int] = None,
                      rope: Optional[tuple] = None, keep_first: int = 0, head_pages: int = 0,
                      gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                     chunk: int = 0) -> torch.Tensor:
+                     chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One token per sequence over the bf16 cache; all heads of a group share one pass over
     the keys and values.  mma: the tensor-core kernel (head sizes 64 and 128; the default
     where it fits) or the CUDA-core one (any head size that is a multiple of 16).
     rope = (k, v, inv_freq, rotary_dim, pairing), tensor-core kernel only: q, k and v are the
     unrotated projections; the kernel rotates q and k and writes k and v into the cache itself
     (k and v None: it reads another run's cache and only rotates q).
-    keep_first, head_pages, gate, sink, sink_values, chunk (CUDA-core kernel only): as attention_generic."""
+    keep_first, head_pages, gate, sink, sink_values, chunk, slopes (CUDA-core kernel only): as attention_generic."""
+    _check_slopes(slopes, n_heads)
     _cuda(q, out, seq_of, pos, table, kcache, vcache, gate, sink_values)
     assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == n_heads and sink_values.is_contiguous())
     sink = bool(sink) or sink_values is not None
-    kept = bool(keep_first or head_pages or gate is not None or sink or chunk)
+    kept = bool(keep_first or head_pages or gate is not None or sink or chunk or slopes is not None)
     assert not kept or (mma is False and rope is None)
     assert gate is None or gate.dtype == torch.bfloat16
     per_head = _gate_per_head(gate, out, n_heads)
@@ -1004,7 +1071,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_head
              ptr(seq_of), ptr(pos), ptr(table), table.shape[1], ring_pages, ptr(kcache), ptr(vcache), int(window or 0),
              float(scale), splits, ptr(scratch), ptr(counters), 0 if counters is None else counters.numel(), int(head_pages),
              int(keep_first or 0), ptr(gate), 0 if gate is None else gate.stride(0), int(per_head), int(bool(sink)),
-             ptr(sink_values), int(chunk or 0), stream_ptr())
+             ptr(sink_values), int(chunk or 0), ptr(slopes), stream_ptr())
         return out
     call(entry, ptr(q), q.stride(0), ptr(out), out.stride(0), T, n_heads, n_kv_heads, head_dim,
          ptr(seq_of), ptr(pos), ptr(table), table.shape[1], ring_pages, ptr(kcache), ptr(vcache), int(window or 0),
@@ -1039,12 +1106,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
                       table: torch.Tensor, ring_pages: int, kcache: torch.Tensor, vcache: torch.Tensor, window: int,
                       scale: float, tc: Optional[bool] = None, exact: bool = False, keep_first: int = 0, head_pages: int = 0,
                       gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                      chunk: int = 0) -> torch.Tensor:
+                      chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Many tokens per sequence over the bf16 cache (which already holds their keys and
     values), flash style.  tc: both products on tcgen05 with S and PV in TMEM (the default where it
     fits), else on mma.sync; both take head sizes 64 and 128.  exact (mma.sync kernel only): the
     attention weights stay 32-bit, split into three bfloat16 terms for the product with the values.
-    keep_first, head_pages, gate, sink, sink_values, chunk (mma.sync kernel only): as attention_generic."""
+    keep_first, head_pages, gate, sink, sink_values, chunk, slopes (mma.sync kernel only; slopes with exact): as
+    attention_generic."""
+    _check_slopes(slopes, n_heads)
     _cuda(q, out, tiles, cu, starts, qlens, table, kcache, vcache, gate, sink_values)
     assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == n_heads and sink_values.is_contiguous())
     sink = bool(sink) or sink_values is not None
@@ -1052,7 +1121,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
     per_head = _gate_per_head(gate, out, n_heads)
     assert q.stride(1) == 1 and out.stride(1) == 1 and out.shape == (q.shape[0], n_heads * head_dim)
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and kcache.dtype == torch.bfloat16
-    plain = not (exact or keep_first or head_pages or gate is not None or sink or chunk)
+    plain = not (exact or keep_first or head_pages or gate is not None or sink or chunk or slopes is not None)
     if tc is None:
         tc = attention_prefill_tc_supported(q, kcache, head_dim) and plain
     assert not tc or plain
@@ -1065,7 +1134,8 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
     call("gb_attention_prefill", ptr(q), q.stride(0), ptr(out), out.stride(0), n_heads, n_kv_heads, head_dim, ptr(tiles),
          tiles.numel() // 2, ptr(cu), ptr(starts), ptr(qlens), ptr(table), table.shape[1], ring_pages, ptr(kcache),
          ptr(vcache), int(window or 0), float(scale), int(bool(exact)), int(head_pages), int(keep_first or 0), ptr(gate),
-         0 if gate is None else gate.stride(0), int(per_head), int(bool(sink)), ptr(sink_values), int(chunk or 0), stream_ptr())
+         0 if gate is None else gate.stride(0), int(per_head), int(bool(sink)), ptr(sink_values), int(chunk or 0),
+         ptr(slopes), stream_ptr())
     return out
 
 

@@ -34,8 +34,8 @@ class Layer:
             FEED_FORWARDS.get(spec.feed_forward.kind)(spec.feed_forward, dtype, device)
         self.norms = {name: NORMS.get(s.kind)(s, dtype, device) for name, s in spec.norms.items()}
         self.extras = {name: EXTRAS.get(s.kind)(s, dtype, device) for name, s in spec.extras.items()}
-        # an arrangement that knows no extra parts is built as before
-        more = {"extras": self.extras} if self.extras else {}
+        # an arrangement that knows no extra parts or constants is built without them
+        more = {**({"extras": self.extras} if self.extras else {}), **spec.block_params}
         self.block = BLOCKS.get(spec.block)(self.mixer, self.feed_forward, self.norms, **more)
 
     def parts(self):
@@ -154,15 +154,16 @@ class Decoder:
 
     def run_views(self, cache: Cache) -> List[RunView]:
         views = []
+        read = {run.cache_of for run in self.spec.schedule if run.cache_of is not None}
         for r, run in enumerate(self.spec.schedule):
             src = r if run.cache_of is None else run.cache_of
             if src in cache.group_of_run:
                 gi, i = cache.group_of_run[src]
                 g = cache.groups[gi]
                 views.append(RunView(r, run.layer, run.cache_of is None, gi, g.k[i], None if g.v is None else g.v[i], g.ring_pages,
-                                      g.spec, g.head_pages, run.add_input))
+                                      g.spec, g.head_pages, run.add_input, src, r in read))
             else:
-                views.append(RunView(r, run.layer, False, add_input=run.add_input))
+                views.append(RunView(r, run.layer, False, add_input=run.add_input, source=r))
         return views
 
     # ---------------------------------------------------------------- forward

@@ -142,7 +142,7 @@ _SIGNATURES = {
     "gb_zero_rows": [_P, _P, _I, _I, _P],
     "gb_gemm_generic": [_P, _I, _L, _P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _P],
     "gb_attention_generic": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _F, _I, _I, _P, _I, _L, _I, _I,
-                             _P, _I, _P],
+                             _P, _I, _P, _P],
     "gb_add_dyt": [_P, _P, _I, _I, _L, _P, _I, _I, _P, _P, _I, _F, _P, _I, _I, _P],
     "gb_scale": [_P, _L, _F, _P],
     "gb_short_conv_silu": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _L, _P],
@@ -158,7 +158,7 @@ _SIGNATURES = {
     "gb_add_rmsnorm_pair": [_P, _P, _I, _P, _I, _P, _I, _I, _P, _I, _I, _P, _P, _I, _F, _F, _P, _P, _I, _I, _P],
     "gb_embed_bigram": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _F, _P, _P, _P],
     "gb_norm_residual_add": [_P, _P, _I, _L, _I, _I, _P, _I, _F, _P, _P],
-    "gb_head_prep_kv_write": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _I, _I, _P, _L, _F, _P, _L, _P, _P, _P,
+    "gb_head_prep_kv_write": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _I, _I, _P, _L, _F, _P, _L, _F, _I, _P, _P, _P,
                               _I, _I, _I, _P, _P, _I, _P],
     "gb_gla": [_P, _P, _P, _I, _L, _P, _I, _L, _P, _I, _F, _F, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
     "gb_gla_segment_floats": [_I, _I, _I, _I, _I],
@@ -177,17 +177,19 @@ _SIGNATURES = {
     "gb_moe_grouped": [_P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _P],
     "gb_glu_clamped": [_P, _L, _P, _I, _I, _I, _F, _P],
     "gb_qk_norm_kv_write": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P, _P, _I, _I, _P, _P, _I, _P],
-    "gb_latent_prep": [_P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _L, _I, _I, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P],
+    "gb_latent_prep": [_P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _L, _I, _I, _P, _P, _P, _P, _I, _I, _P, _I, _I, _F, _P],
     "gb_selective_scan": [_P, _L, _P, _L, _I, _P, _I, _L, _I, _I, _P, _L, _P, _P, _P, _P, _P, _L, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     "gb_selective_scan_segment_floats": [_I, _I, _I, _I],
     "gb_norm_sandwich": [_P, _P, _I, _L, _P, _I, _L, _P, _P, _F, _P, _P, _I, _F, _P, _I, _P, _P, _I, _I, _P],
+    "gb_layernorm": [_P, _P, _I, _L, _P, _P, _P, _I, _F, _P, _I, _F, _P, _I, _I, _P, _I, _P, _I, _P],
+    "gb_rms_rows": [_P, _I, _L, _I, _I, _P, _I, _F, _P, _I, _L, _P],
     "gb_token_side_gate": [_P, _I, _L, _P, _I, _L, _I, _P, _I, _I, _I, _I, _P, _I, _L, _P],
     "gb_pack_latent_heads": [_P, _L, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P],
     "gb_latent_decode_supported": [_I, _I, _I, _I, _I],
     "gb_latent_decode_set_mma": [_I],
     "gb_latent_decode_scratch_floats": [_I, _I, _I, _I],
     "gb_latent_decode": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _F, _I, _P, _I, _P, _P, _L, _P],
-    "gb_head_matmul": [_P, _I, _L, _I, _P, _I, _I, _I, _I, _P, _I, _L, _I, _I, _P],
+    "gb_head_matmul": [_P, _I, _L, _I, _P, _I, _I, _I, _I, _P, _I, _L, _I, _I, _P, _I, _L, _P],
     "gb_sample": [_P, _L, _I, _I, _P, _P, _F, _I, _F, _F, _P, _P, _P, _P],
     "gb_gemm_tc": [_P, _L, _P, _L, _P, _I, _P, _I, _L, _I, _I, _I, _P, _P, _I, _I, _I, _P],
     "gb_gemm_tc_tile": [_I],
@@ -199,7 +201,7 @@ _SIGNATURES = {
     "gb_gemm_tc_supported": [_P, _L, _P, _L, _I],
     "gb_attention_decode": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _P],
     "gb_attention_decode_kept": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _I, _I, _P, _L, _I, _I,
-                                 _P, _I, _P],
+                                 _P, _I, _P, _P],
     "gb_attention_decode_mma": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _P],
     "gb_attention_decode_mma_rope": [_P, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I,
                                      _P, _P, _I, _P],
@@ -210,7 +212,7 @@ _SIGNATURES = {
     "gb_gemm_tc_set_stamps": [_P, _I, _I],
     "gb_attention_decode_scratch_floats": [_I, _I, _I, _I],
     "gb_attention_decode_supported": [_I, _I, _I],
-    "gb_attention_prefill": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _I, _I, _P, _I, _P],
+    "gb_attention_prefill": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _I, _I, _P, _I, _P, _P],
     "gb_attention_prefill_supported": [_I, _I, _I],
     "gb_attention_prefill_tile": [],
     "gb_attention_prefill_tc": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _L, _I, _F, _P],

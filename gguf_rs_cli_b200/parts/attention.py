@@ -32,6 +32,12 @@ the sequence's start, a token seeing the earlier tokens of its own chunk only (i
 ring of that many positions); a sink whose score is a learned number per head, not scaled (`sink="learned"`, tensor
 `sink` [heads]); `exact=True` asks for 32-bit scores and weights where nothing else does.  These paths also take q/k/v
 biases and `shares_kv` (the layer then prepares its queries only and attends to the other run's keys and values).
+
+And for designs without a rotation whose keys are also their values: a bias that grows with the distance (`distance_bias`
+= e: head h of H loses 2^(-e (h+1)/H) times the distance of query and key from every scaled score); values that are the
+keys as projected, bias included, before their norm (`values="keys"`: no v matrix, the cache holds the normed key and the
+bare one); the query temperature beside a head norm; biases on chosen projections (`bias` a sequence of names, "o" among
+them).
 """
 from __future__ import annotations
 
@@ -50,14 +56,15 @@ from .registry import register_mixer
 @register_mixer("attention")
 class Attention(Part):
     """params: hidden_size, num_heads, num_kv_heads, head_dim, scale, window (None or W),
-    bias (q/k/v biases), shares_kv (default False), v_head_dim (default head_dim),
+    bias (True: q/k/v biases; or the names that have one, of q, k, v, o), shares_kv (default False), v_head_dim (default head_dim),
     qk_norm_eps (default None: no normalisation), q_temp (default None, or {"coef", "every"}),
     head_norm_eps (default None), keep_first (default 0), out_gate (default False), v_mix (None, "gives" or "takes"),
     v_mix_optional (the folder may hold the scalar although nothing is mixed), conv (default None; taps of a short
     convolution on q, k and v), sink (default False; "learned": a score per head from the tensor `sink`), out_gate "head":
     one gate per head, chunk (None or C: chunks of C positions in a window's place), exact (default False), cache_span
-    (when present: the positions the cache keeps, None for all, where runs with windows of their own share one cache).
-    tensors: q [nh*hd, E], k [nkv*hd, E], v [nkv*vd, E], o [E, nh*vd], optional q_bias, k_bias, v_bias;
+    (when present: the positions the cache keeps, None for all, where runs with windows of their own share one cache),
+    distance_bias (default None; the exponent e), values (default None; "keys").
+    tensors: q [nh*hd, E], k [nkv*hd, E], v [nkv*vd, E], o [E, nh*vd], optional q_bias, k_bias, v_bias, o_bias [E];
     with head_norm_eps q_norm, k_norm [hd]; with out_gate g [nh*vd, E] ("head": [nh, E]); with v_mix the scalar v_mix;
     with conv q_conv, k_conv, v_conv [channels, taps]."""
 
@@ -89,27 +96,42 @@ class Attention(Part):
         self.chunk = int(p.get("chunk") or 0)
         if self.chunk and (self.window or p.get("keep_first")):
             raise ValueError("attention: chunks go with neither a window nor kept first positions")
+        bias = p.get("bias") or ()
+        self.biased = ("q", "k", "v") if bias is True else tuple(bias)
+        if any(n not in ("q", "k", "v", "o") for n in self.biased):
+            raise ValueError(f"attention: bias {bias!r} names projections that are not q, k, v, o")
+        self.distance_bias = float(p.get("distance_bias") or 0.0)
+        self.keys_are_values = p.get("values") == "keys"
+        if p.get("values") not in (None, "keys"):
+            raise ValueError(f"attention: values {p.get('values')!r} is not None or 'keys'")
+        if self.keys_are_values and (self.vd != self.hd or self.conv > 1 or p.get("v_mix") or self.shares_kv or "v" in self.biased):
+            raise ValueError("attention: values that are the keys have the keys' size and go with neither a convolution, mixed "
+                             "values, a bias of their own nor shares_kv")
+        if position is not None and getattr(position, "gain", 1.0) != 1.0:
+            raise ValueError("attention: a rotation whose sine and cosine carry a factor is not supported here")
         self.v_mix = p.get("v_mix") or None
         if self.v_mix not in (None, "gives", "takes"):
             raise ValueError(f"attention: v_mix {self.v_mix!r} is not one of None, 'gives', 'takes'")
         # heads with a norm of their own, a gate, kept first positions or mixed values: prepared by one kernel
         # (norm, rotation, mixing, cache write) and attended to with 32-bit weights
         self.prepared = bool(self.head_norm_eps is not None or self.keep_first or self.out_gate or self.v_mix or self.conv > 1
-                             or self.sink or self.chunk or p.get("exact"))
+                             or self.sink or self.chunk or self.distance_bias or self.keys_are_values or "o" in self.biased or p.get("exact"))
         # where the parts of the fused projection start: q, k, v and the gate, each at a multiple of 8 rows
         self.off, rows = {}, 0
         own = 0 if self.shares_kv else 1
-        for n, size in (("q", self.nh * self.hd), ("k", own * self.nkv * self.hd), ("v", own * self.nkv * self.vd),
+        for n, size in (("q", self.nh * self.hd), ("k", own * self.nkv * self.hd), ("v", 0 if self.keys_are_values else own * self.nkv * self.vd),
                         ("g", (self.nh if self.gate_per_head else self.nh * self.vd) if self.out_gate else 0)):
             self.off[n] = (rows + 7) // 8 * 8
             rows = self.off[n] + size
         self.gate_rows = rows - self.off["g"]
+        if self.keys_are_values:
+            self.off["v"] = self.off["k"]
         self.conv_channels = self.off["v"] + own * self.nkv * self.vd      # q, k, v and the empty rows between them
         # normalised q and k, a query temperature or values of their own size: the exact path
         self.exact = self.prepared or self.vd != self.hd or self.qk_norm_eps is not None or self.temp_coef != 0.0
-        if self.prepared and (self.qk_norm_eps is not None or self.temp_coef != 0.0):
-            raise ValueError("attention: head_norm_eps, keep_first, out_gate, v_mix, conv, sink, chunk and exact go with neither "
-                             "qk_norm_eps nor q_temp")
+        if self.prepared and self.qk_norm_eps is not None:
+            raise ValueError("attention: qk_norm_eps goes with none of head_norm_eps, keep_first, out_gate, v_mix, conv, sink, chunk, "
+                             "distance_bias, values, a bias on o and exact")
         if self.shares_kv and self.v_mix:
             raise ValueError("attention: a layer that reads another's keys and values has no values to mix")
         if self.exact and not self.prepared and (position is not None or self.shares_kv):
@@ -128,14 +150,18 @@ class Attention(Part):
     def state_spec(self) -> Dict[str, Tuple[Tuple[int, ...], str]]:
         return {"conv": ((self.conv - 1, self.conv_channels), "float32")} if self.conv > 1 else {}
 
+    def _projections(self) -> List[str]:
+        """The projections of the mixer's input that this layer has, without the gate."""
+        return ["q"] + ([] if self.shares_kv else ["k"] if self.keys_are_values else ["k", "v"])
+
     def tensor_requests(self) -> List[TensorRequest]:
         E, t = self.p["hidden_size"], self.spec.tensors
-        names = ["q"] + ([] if self.shares_kv else ["k", "v"])
+        names = self._projections()
         rows = {"q": self.nh * self.hd, "k": self.nkv * self.hd, "v": self.nkv * self.vd}
         req = [TensorRequest(t[n], (rows[n], E)) for n in names]
         req.append(TensorRequest(t["o"], (E, self.nh * self.vd)))
-        if self.p.get("bias"):
-            req += [TensorRequest(t[n + "_bias"], (rows[n],)) for n in names]
+        rows["o"] = E
+        req += [TensorRequest(t[n + "_bias"], (rows[n],)) for n in names + ["o"] if n in self.biased]
         if self.head_norm_eps is not None:
             req += [TensorRequest(t["q_norm"], (self.hd,), init="ones"), TensorRequest(t["k_norm"], (self.hd,), init="ones")]
         if self.out_gate:
@@ -153,12 +179,14 @@ class Attention(Part):
         t = self.spec.tensors
         if self.prepared:
             return self._load_prepared(store, req)
-        names = ["q"] + ([] if self.shares_kv else ["k", "v"])
+        names = self._projections()
         mats = [store.get(req[t[n]]) for n in names]
         dt = mats[0].dtype
         w = torch.cat([m.to(dt) for m in mats], dim=0) if len(mats) > 1 else mats[0]
         b = None
-        if self.p.get("bias"):
+        if self.biased:
+            if any(n not in self.biased for n in names):
+                raise ValueError("attention: this path takes biases on all of q, k and v or on none")
             b = torch.cat([store.get(req[t[n + "_bias"]]).to(torch.float32) for n in names], dim=0)
         self.qkv = Linear(w, b, name="attn.qkv")
         self.o = Linear(store.get(req[t["o"]]), name="attn.o")
@@ -167,15 +195,15 @@ class Attention(Part):
         """q, k, v and the gate as one matrix, each part starting at a multiple of 8 rows (zero rows between), so that
         one product reads h once and every slice of its result is aligned."""
         t = self.spec.tensors
-        names = ["q"] + ([] if self.shares_kv else ["k", "v"]) + (["g"] if self.out_gate else [])
+        names = self._projections() + (["g"] if self.out_gate else [])
         mats = [store.get(req[t[n]]) for n in names]
         dt = mats[0].dtype
         total = (self.off["g"] + self.gate_rows + 7) // 8 * 8
         bias = None
-        if self.p.get("bias"):
+        if any(n in self.biased for n in names):
             bias = torch.zeros(total, dtype=torch.float32, device=mats[0].device)
             for n in names:
-                if n != "g":
+                if n in self.biased:
                     b = store.get(req[t[n + "_bias"]])
                     bias[self.off[n]:self.off[n] + b.numel()] = b.to(torch.float32)
         self.sink_values = store.get(req[t["sink"]]).to(torch.float32).contiguous() if self.sink_learned else None
@@ -190,7 +218,12 @@ class Attention(Part):
         if pad:
             parts.append(torch.zeros(pad, mats[0].shape[1], dtype=dt, device=mats[0].device))
         self.qkv = Linear(torch.cat(parts, dim=0).contiguous(), bias, name="attn.qkvg")
-        self.o = Linear(store.get(req[t["o"]]), name="attn.o")
+        o_bias = store.get(req[t["o_bias"]]).to(torch.float32).contiguous() if "o" in self.biased else None
+        self.o = Linear(store.get(req[t["o"]]), o_bias, name="attn.o")
+        self.slopes = None
+        if self.distance_bias:
+            slopes = [2.0 ** (-self.distance_bias * (h + 1) / self.nh) for h in range(self.nh)]
+            self.slopes = torch.tensor(slopes, dtype=torch.float64).to(torch.float32).to(mats[0].device)
         self.q_norm = self.k_norm = None
         if self.head_norm_eps is not None:
             self.q_norm, self.k_norm = store.get(req[t["q_norm"]]), store.get(req[t["k_norm"]])
@@ -290,12 +323,12 @@ class Attention(Part):
         kernels.head_prep_kv_write(q, k, v, nh, nkv, hd, vd, self.q_norm, self.k_norm, self.head_norm_eps or 1.0,
                                    None if pos is None else pos.inv_freq, 0 if pos is None else pos.rotary_dim,
                                    0 if pos is None else pos.pairing, v_first, self.mix, first_out, ctx.seq_of, ctx.pos, table,
-                                   run.ring_pages, run.head_pages, run.k, run.v)
+                                   run.ring_pages, run.head_pages, run.k, run.v, temp_coef=self.temp_coef, temp_every=self.temp_every)
         ctx.mark("heads")
         out = ctx.ws.get("attn.out", (T, nh * vd), ctx.dtype)
         tiles = ctx.plan_of(self).get("tiles")
         kept = dict(keep_first=self.keep_first, head_pages=run.head_pages, gate=gate, sink=self.sink, sink_values=self.sink_values,
-                    chunk=self.chunk)
+                    chunk=self.chunk, slopes=self.slopes)
         if not ctx.decode and tiles is not None and self._exact_tiled() and kernels.attention_prefill_supported(q, run.k, hd):
             # prompts, keys and values of 64 or 128 entries: the tiled kernel with 32-bit weights
             kernels.attention_prefill(q, out, nh, nkv, hd, tiles, ctx.cu, ctx.starts, ctx.qlens, table, run.ring_pages,

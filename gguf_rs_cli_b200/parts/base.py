@@ -111,6 +111,8 @@ class RunView:
     kv_spec: Optional[KVSpec] = None
     head_pages: int = 0           # table entries in front of the ring: pages of first positions that are kept for ever
     add_input: bool = False       # the embedding's result is added to the stream once more before this run
+    source: Optional[int] = None  # the run whose cache this one reads (its own number where it owns its cache)
+    has_readers: bool = False     # a later run reads this run's cache
 
 
 @dataclass
@@ -198,6 +200,16 @@ class Blend:
     weights: Tuple[torch.Tensor, torch.Tensor]
     mix: float
     eps: float
+
+
+@dataclass
+class RoutedRows:
+    """What a mixture hands over unsummed to a block whose next kernel can finish it: token t's term is base[t] (None: nothing)
+    plus sum_r weights[t, r] rows[place_of[t * top + r]] (place_of None: the pairs' own order), the choices in their order."""
+    base: Optional[torch.Tensor]         # float32 [T, E]
+    rows: torch.Tensor                   # float32 [T * top, E]
+    weights: torch.Tensor                # float32 [T, top]
+    place_of: Optional[torch.Tensor] = None
 
 
 @dataclass

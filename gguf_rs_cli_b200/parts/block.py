@@ -8,6 +8,18 @@ from .base import RunView, StepContext, Stream
 from .registry import register_block
 
 
+def own_rows(stream: Stream, ctx: StepContext):
+    """x as the products of sublayers that read the stream itself take it: x in 32-bit mode, else its bfloat16 copy."""
+    if stream.pending is not None:
+        raise RuntimeError("a term is pending on the stream; an arrangement whose sublayers read x adds every term at once")
+    if ctx.dtype == torch.float32:
+        return stream.x
+    if stream.xb is None:
+        stream.xb = ctx.ws.get("stream.xb", stream.x.shape, torch.bfloat16)
+        kernels.norm_residual_add(stream.x, None, None, 1.0, xb=stream.xb)
+    return stream.xb
+
+
 @register_block("prenorm")
 class PreNormBlock:
     """x += mixer(norm_m(x)); x += ff(norm_f(x)) (src/model/llama.rs:361-404).  The sums
@@ -79,30 +91,49 @@ class OutputNormBlock:
                 raise ValueError(f"outnorm: the norm of kind {norms[name].spec.kind!r} cannot norm a sublayer's result into the stream")
 
     def forward(self, stream: Stream, ctx: StepContext, run: RunView) -> None:
-        term = self.mixer.forward(self._rows(stream, ctx), ctx, run)
+        term = self.mixer.forward(own_rows(stream, ctx), ctx, run)
         self.norms["mixer"].add_normed(stream, term, ctx)
         ctx.mark("mixer_norm")
         if self.feed_forward is None:
             return
         if getattr(self.feed_forward, "reads_stream", False):
             # a part that decides in 32-bit (a router) also gets the stream itself, not only its bfloat16 copy
-            term = self.feed_forward.forward(self._rows(stream, ctx), ctx, x32=stream.x)
+            term = self.feed_forward.forward(own_rows(stream, ctx), ctx, x32=stream.x)
         else:
-            term = self.feed_forward.forward(self._rows(stream, ctx), ctx)
+            term = self.feed_forward.forward(own_rows(stream, ctx), ctx)
         self.norms["feed_forward"].add_normed(stream, term, ctx)
         ctx.mark("ff_norm")
 
-    @staticmethod
-    def _rows(stream: Stream, ctx: StepContext):
-        """x as the sublayers' products read it: x itself in 32-bit mode, else its bfloat16 copy."""
-        if stream.pending is not None:
-            raise RuntimeError("outnorm: a term is pending on the stream; this arrangement adds every term at once")
-        if ctx.dtype == torch.float32:
-            return stream.x
-        if stream.xb is None:
-            stream.xb = ctx.ws.get("stream.xb", stream.x.shape, torch.bfloat16)
-            kernels.norm_residual_add(stream.x, None, None, 1.0, xb=stream.xb)
-        return stream.xb
+
+@register_block("postnorm")
+class PostNormBlock:
+    """x <- norm_m(alpha x + mixer(x)); x <- norm_f(alpha x + ff(x)): the norms stand behind the sums, the sublayers read x
+    itself.  One kernel per sublayer takes the sum, norms it and writes the new x (32-bit) with its bfloat16 copy, which the
+    next sublayer's products read; a mixture's weighted sum over its experts' rows is part of the same pass.  alpha: a
+    constant factor of x in the sum (default 1)."""
+
+    norm_names = ("mixer", "feed_forward")
+    graph_class = ()
+
+    def __init__(self, mixer, feed_forward, norms, alpha: float = 1.0):
+        self.mixer, self.feed_forward, self.norms, self.alpha = mixer, feed_forward, norms, float(alpha)
+        for name in self.norm_names[:1 if feed_forward is None else 2]:
+            if name not in norms or not hasattr(norms[name], "norm_sum"):
+                raise ValueError(f"postnorm: the layer needs a norm {name!r} that can norm the sum of the stream and a term")
+
+    def forward(self, stream: Stream, ctx: StepContext, run: RunView) -> None:
+        term = self.mixer.forward(own_rows(stream, ctx), ctx, run)
+        self.norms["mixer"].norm_sum(stream, term, ctx, self.alpha)
+        ctx.mark("mixer_norm")
+        if self.feed_forward is None:
+            return
+        rows, ff = own_rows(stream, ctx), self.feed_forward
+        if getattr(ff, "reads_stream", False):
+            term = ff.forward(rows, ctx, x32=stream.x, unsummed=True)
+        else:
+            term = ff.forward(rows, ctx)
+        self.norms["feed_forward"].norm_sum(stream, term, ctx, self.alpha)
+        ctx.mark("ff_norm")
 
 
 @register_block("parallel")

@@ -11,7 +11,7 @@ from .. import kernels
 from ..weights.loader import TensorRequest, WeightStore
 from typing import Optional
 
-from .base import DeferredNorm, Part, StepContext
+from .base import DeferredNorm, Part, RoutedRows, StepContext
 from .linear import Linear
 from .registry import register_feed_forward
 
@@ -116,8 +116,12 @@ class RoutedExperts(Part):
     `identity` experts without matrices, numbered behind the others, whose result is the token's own row h (the router's
     matrix and the correction then have experts + identity rows).
 
-    params: hidden_size, experts, top, groups, keep, scale, expert_ff, limit, shared_ff, shared_limit (None: no shared
-    expert), score ("sigmoid" or "softmax"), correction (default False), identity (default 0).  tensors: router
+    With limit None the unit is the plain silu(g) u (shared_limit likewise for the shared expert, whose gate and up then run
+    as one product with the unit in its epilogue).  A block whose next kernel can finish the weighted sum asks for the
+    experts' rows unsummed (RoutedRows).
+
+    params: hidden_size, experts, top, groups, keep, scale, expert_ff, limit, shared_ff (None: no shared expert), shared_limit,
+    score ("sigmoid" or "softmax"), correction (default False), identity (default 0).  tensors: router
     [experts + identity, E]; experts: the prefix of the experts' names (<prefix><i>.gate [F, E], .up [F, E], .down [E, F]);
     shared: the prefix of the shared expert's (.gate, .up [Fs, E], .down [E, Fs]); correction [experts + identity]."""
 
@@ -127,6 +131,8 @@ class RoutedExperts(Part):
         self.n, self.top, self.F = int(p["experts"]), int(p["top"]), int(p["expert_ff"])
         self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or 1)
         self.shared_ff = p.get("shared_ff")
+        # the kernels' convention: 0 is the unit without limits
+        self.limit, self.shared_limit = float(p.get("limit") or 0.0), float(p.get("shared_limit") or 0.0)
         self.identity = int(p.get("identity") or 0)
         self.n_all = self.n + self.identity
         self.score = p.get("score", "sigmoid")
@@ -168,7 +174,11 @@ class RoutedExperts(Part):
         self.correction = store.get(req[-1]).to(torch.float32).contiguous() if self.corrected else None
         if self.shared_ff:
             g, u, d = (store.get(r) for r in req[1 + 3 * self.n:4 + 3 * self.n])
-            self.shared_gate_up = Linear(torch.cat([g, u.to(g.dtype)], dim=0), name="moe.shared_gate_up")
+            self.shared_tiles = None
+            if not self.shared_limit and g.dtype == torch.bfloat16 and self.p["hidden_size"] % 8 == 0 and g.is_cuda:
+                self.shared_tiles = kernels.interleave_gate_up(g, u.to(g.dtype))
+            else:
+                self.shared_gate_up = Linear(torch.cat([g, u.to(g.dtype)], dim=0), name="moe.shared_gate_up")
             self.shared_down = Linear(d, name="moe.shared_down")
 
     TOKEN_BY_TOKEN = 16           # steps of at most this many tokens run every (token, choice) pair for itself
@@ -177,7 +187,19 @@ class RoutedExperts(Part):
     graph_class = ()              # grids depend on the number of tokens only
     reads_stream = True           # a block that has the rows in 32-bit gives them too (x32): the router reads those
 
-    def forward(self, h, ctx: StepContext, x32: Optional[torch.Tensor] = None) -> torch.Tensor:
+    def _shared(self, h, ctx: StepContext) -> torch.Tensor:
+        act = ctx.ws.get("moe.shared_act", (h.shape[0], int(self.shared_ff)), ctx.dtype)
+        if self.shared_limit:
+            kernels.glu_clamped(self.shared_gate_up(h, ctx), act, self.shared_limit)
+        elif self.shared_tiles is not None and kernels.gemm_tc_supported(h, self.shared_tiles):
+            kernels.gemm_tc(h, self.shared_tiles, None, act, swiglu_features=int(self.shared_ff))
+        elif self.shared_tiles is not None:
+            raise RuntimeError("moe: the activations given do not fit the fused product the shared expert was loaded for")
+        else:
+            kernels.swiglu(self.shared_gate_up(h, ctx), act)
+        return self.shared_down(act, ctx, out_dtype=torch.float32, buffer="moe.out")
+
+    def forward(self, h, ctx: StepContext, x32: Optional[torch.Tensor] = None, unsummed: bool = False):
         T, E, top = h.shape[0], self.p["hidden_size"], self.top
         # the router's product in 32-bit sums, from 32-bit rows where the block has them, and its choice
         ids = ctx.ws.get("moe.ids", (T, top), torch.int32)
@@ -187,26 +209,30 @@ class RoutedExperts(Part):
         ctx.mark("router")
         out = ctx.ws.get("moe.out", (T, E), torch.float32)
         if self.shared_ff:
-            Fs = int(self.shared_ff)
-            act = kernels.glu_clamped(self.shared_gate_up(h, ctx), ctx.ws.get("moe.shared_act", (T, Fs), ctx.dtype),
-                                      float(self.p["shared_limit"]))
-            self.shared_down(act, ctx, out_dtype=torch.float32, buffer="moe.out")
+            self._shared(h, ctx)
             ctx.mark("shared")
+        # rows that the caller sums: no identity experts among them, whose rows are the tokens' own
+        unsummed = unsummed and not self.identity
+        base, place_of = out if self.shared_ff else None, None
+        if unsummed:
+            out = None
         if not ctx.decode and T * top >= self.BY_EXPERT * self.n and self.F * E >= self.BY_EXPERT_ENTRIES \
                 and kernels.moe_grouped_supported(h, self.w_gate):
             # very many tokens (an expert gets 128 rows or more on average) and large experts: every expert's products on
             # the tcgen05 kernels (8,192 pairs, 16 experts of 3,584 x 4,096: 1.65 against 3.99 ms; of 2,048 x 2,048: 1.17
             # against 1.21 ms, the launches of small products fill a quarter of the device)
-            kernels.moe_by_expert(h, ids, weights, self.w_gate, self.w_up, self.w_down, float(self.p["limit"]), out, ctx,
-                                  accumulate=bool(self.shared_ff), identity=self.identity)
+            got = kernels.moe_by_expert(h, ids, weights, self.w_gate, self.w_up, self.w_down, self.limit, out, ctx,
+                                        accumulate=bool(self.shared_ff), identity=self.identity)
+            if unsummed:
+                got, place_of = got
         elif T > self.TOKEN_BY_TOKEN and kernels.moe_grouped_supported(h, self.w_gate):
             # many tokens: pairs sorted by expert on the device, tiles of 64 pairs on the tensor cores
-            kernels.moe_grouped(h, ids, weights, self.w_gate, self.w_up, self.w_down, float(self.p["limit"]), out, ctx,
-                                accumulate=bool(self.shared_ff), identity=self.identity)
+            got = kernels.moe_grouped(h, ids, weights, self.w_gate, self.w_up, self.w_down, self.limit, out, ctx,
+                                      accumulate=bool(self.shared_ff), identity=self.identity)
         else:
             y = ctx.ws.get("moe.units", (T, top, self.F), ctx.dtype)
-            kernels.moe_gate_up(h, ids, self.w_gate, self.w_up, float(self.p["limit"]), y, identity=self.identity)
-            kernels.moe_down(y, ids, weights, self.w_down, out, accumulate=bool(self.shared_ff), ws=ctx.ws, identity=self.identity,
-                             h=h)
+            kernels.moe_gate_up(h, ids, self.w_gate, self.w_up, self.limit, y, identity=self.identity)
+            got = kernels.moe_down(y, ids, weights, self.w_down, out, accumulate=bool(self.shared_ff), ws=ctx.ws,
+                                   identity=self.identity, h=h)
         ctx.mark("experts")
-        return out
+        return RoutedRows(base, got, weights, place_of) if unsummed else out

@@ -9,7 +9,7 @@ import torch
 
 from .. import kernels
 from ..weights.loader import TensorRequest, WeightStore
-from .base import FUSE_MAX_TOKENS, Blend, DeferredNorm, Part, StepContext, Stream
+from .base import FUSE_MAX_TOKENS, Blend, DeferredNorm, Part, RoutedRows, StepContext, Stream
 from .registry import register_norm
 
 
@@ -152,4 +152,40 @@ class DynamicTanh(Part):
             if stream.pending is not None:
                 stream.drop_shadow()
             stream.pending = None
+        return out
+
+
+@register_norm("layernorm")
+class LayerNorm(Part):
+    """Layer norm with a weight and no bias: (x - mean) / sqrt(variance + eps) * w, the variance being the mean of the
+    squared deviations; all in 32-bit.  params: size, eps.  tensors: weight [size]."""
+
+    graph_class = ()
+
+    def tensor_requests(self) -> List[TensorRequest]:
+        return [TensorRequest(self.spec.tensors["weight"], (self.p["size"],), init="ones")]
+
+    def load(self, store: WeightStore) -> None:
+        self.weight = store.get(self.tensor_requests()[0])
+
+    def norm_sum(self, stream: Stream, term, ctx: StepContext, alpha: float = 1.0) -> None:
+        """x <- LN(alpha x + term); in bfloat16 mode the same kernel renews the stream's bfloat16 copy.  term: rows [T, size],
+        or a mixture's RoutedRows, whose weighted sum then runs in the same pass."""
+        if stream.pending is not None or stream.more:
+            raise RuntimeError("layernorm: a term is pending on the stream")
+        xb = ctx.ws.get("stream.xb", stream.x.shape, torch.bfloat16) if ctx.dtype == torch.bfloat16 else None
+        y, routed = term, None
+        if isinstance(term, RoutedRows):
+            y, routed = term.base, (term.rows, term.weights, term.place_of)
+        kernels.layernorm(stream.x, y, self.weight, self.p["eps"], alpha=alpha, routed=routed, xb=xb)
+        stream.xb, stream.ssq, stream.ssq_parts = xb, None, 0
+
+    def apply(self, stream: Stream, ctx: StepContext, rows: Optional[torch.Tensor] = None, buffer: str = "normed",
+              absorbed: bool = False):
+        """LN(x) of all rows, or of `rows` only; x is left as it is."""
+        if stream.pending is not None or stream.more:
+            raise RuntimeError("layernorm: this norm adds no pending term; it follows blocks that add every term at once")
+        n = stream.x.shape[0] if rows is None else rows.numel()
+        out = ctx.ws.get(buffer, (n, self.p["size"]), ctx.dtype)
+        kernels.layernorm(stream.x, None, self.weight, self.p["eps"], rows=rows, h=out, write_x=False)
         return out
