@@ -4,7 +4,7 @@ one B200.  Prints one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--layers L] [--batch B] [--no-points] [--prompt-steps 128,256] [--shape 8b|1b|13b]
-                    [--design debonex|dilalix|nazerax|fomodra [--sizes 1b,8b]]
+                    [--design debonex|dilalix|nazerax|fomodra|betirax [--sizes 1b,8b]]
 
 `value` is decoded tokens a second at batch 8 after 512-token prompts, timed on the
 device with CUDA events around K decode steps (each step: index arrays host to
@@ -382,10 +382,33 @@ def fomodra_config(z):
             "layers": [layer(i) for i in range(z["layers"])]}
 
 
-DESIGN_CONFIGS = {"debonex": debonex_config, "dilalix": dilalix_config, "nazerax": nazerax_config, "fomodra": fomodra_config}
-# the closest of the other designs (a recurrent rule and attention), which a design is measured beside
-CLOSEST = {"dilalix": ("debonex", debonex_config), "nazerax": ("dilalix-dense", dilalix_dense_config),
-           "fomodra": ("dilalix", dilalix_config)}
+def betirax_config(z):
+    """Attention (window of 1,024, a distance bias, keys as values, a gate per entry) twice, latent attention (queries through a
+    latent of 3/8 of the width, YaRN over 4,096 positions times 4), latent attention on the rows of the layer before; dense
+    feed-forwards and mixtures of 16 experts (4 of them per token, and a shared one: Dilalix's sizes) in turn."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "shared": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 4}}
+    attn = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head"], "vdim": z["head"], "scale": z["head"] ** -0.5,
+            "mask": {"size": 1024}, "q_temp": {"coef": 0.1, "every": 1024}}
+    latent = {"heads": z["heads"], "dim": z["latent_dim"], "rot_dim": z["rot"], "kv_rank": z["kv_rank"], "q_rank": 3 * z["width"] // 8,
+              "vdim": z["head"], "scale": (z["latent_dim"] + z["rot"]) ** -0.5,
+              "rot": {"base": 10000.0, "dims": z["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+
+    def layer(i):
+        mlp = moe if i % 2 else dense
+        if i % 4 < 2:
+            return {"type": "attention", "mixer": attn, "mlp": mlp}
+        return {"type": "latent_attention", "mixer": latent if i % 4 == 2 else {**latent, "kv_from": i - 1}, "mlp": mlp}
+
+    return {"architecture": "Betirax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "postln_alpha": 2.0, "layers": [layer(i) for i in range(z["layers"])]}
+
+
+DESIGN_CONFIGS = {"debonex": debonex_config, "dilalix": dilalix_config, "nazerax": nazerax_config, "fomodra": fomodra_config,
+                  "betirax": betirax_config}
+# the closest of the other designs, which a design is measured beside
+CLOSEST = {"dilalix": [("debonex", debonex_config)], "nazerax": [("dilalix-dense", dilalix_dense_config)],
+           "fomodra": [("dilalix", dilalix_config)], "betirax": [("fomodra", fomodra_config), ("dilalix", dilalix_config)]}
 
 
 def stage_times(llm, lens, starts=0, reps=3):
@@ -445,8 +468,7 @@ def run_design(args, pk):
         z = DESIGN_SIZES[name]
         row = {"config": z}
         arms = [(args.design, DESIGN_CONFIGS[args.design](z))]
-        if args.design in CLOSEST:
-            arms.append((CLOSEST[args.design][0], CLOSEST[args.design][1](z)))
+        arms += [(other, make(z)) for other, make in CLOSEST.get(args.design, [])]
         for arm, raw in arms + [("llama", llama_config(z))]:
             llm = from_random(raw, seed=0, dtype="bfloat16", device="cuda:0")
             torch.cuda.synchronize()
