@@ -92,11 +92,20 @@ __global__ void latent_prep_kernel(const void* __restrict__ q, long long ldq, co
                                    const int* __restrict__ seq_of,
                                    const int* __restrict__ pos, const int* __restrict__ table, int table_width,
                                    int ring_pages, void* __restrict__ cache, int cache_dtype, int halves, float rot_gain) {
+    extern __shared__ float lp_cs[];              // cosines, then sines, of the token's position
     __shared__ float red[32];
     const int t = blockIdx.x;
     const int b = seq_of[t];
     if (b < 0) return;
     const int p = pos[t];
+    const int half = rot_dims / 2, pairs = Rd / 2;          // Rd even: checked by the caller
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf(float(p) * inv_freq[i], &s, &c);
+        lp_cs[i] = c * rot_gain;
+        lp_cs[half + i] = s * rot_gain;
+    }
+    __syncthreads();
     const size_t drow = size_t(t) * size_t(ldd);
     const size_t rrow = size_t(t) * (C + Rd);
     size_t crow = 0;
@@ -120,14 +129,12 @@ __global__ void latent_prep_kernel(const void* __restrict__ q, long long ldq, co
         }
     }
     // rotated parts: item 0 is the shared key part, items 1..H the heads' query parts
-    const int half = rot_dims / 2, pairs = Rd / 2;          // Rd even: checked by the caller
     for (int idx = threadIdx.x + (dkv ? 0 : pairs); idx < (H + 1) * pairs; idx += blockDim.x) {
         const int item = idx / pairs, i = idx - item * pairs;
         float sn = 0.f, cs = 1.f;
         if (i < half) {
-            sincosf(float(p) * inv_freq[i], &sn, &cs);
-            sn *= rot_gain;
-            cs *= rot_gain;
+            cs = lp_cs[i];
+            sn = lp_cs[half + i];
         }
         // the pair that angle i turns: neighbours (2i, 2i+1), or with `halves` entries (i, i + half); pairs behind the
         // rotated entries pass unchanged either way
@@ -168,7 +175,8 @@ GB_API int gb_latent_prep(const void* q, long long ldq, const void* dkv, long lo
     GB_REQUIRE(rot_dims == 0 || inv_freq, "gb_latent_prep: no table of frequencies");
     GB_REQUIRE(!dkv || (table && cache && w && ring_pages > 0 && table_width >= 1 && eps > 0.f), "gb_latent_prep: cache missing");
     if (T == 0) return 0;
-    latent_prep_kernel<<<T, 128, 0, stream>>>(q, ldq, dkv, ldd, dtype, H, D, Rd, C, rot_dims, inv_freq, w, w_dtype, eps, qa, lda,
+    GB_REQUIRE(rot_dims <= 8192, "gb_latent_prep: %d rotated entries are too many", rot_dims);
+    latent_prep_kernel<<<T, 256, size_t(rot_dims) * sizeof(float), stream>>>(q, ldq, dkv, ldd, dtype, H, D, Rd, C, rot_dims, inv_freq, w, w_dtype, eps, qa, lda,
                                               qa_stride, qa_off, row_out, seq_of, pos, table, table_width, ring_pages, cache, cache_dtype, halves, rot_gain);
     GB_LAUNCH_OK("gb_latent_prep");
     return 0;
@@ -203,11 +211,42 @@ __global__ void pack_latent_heads_kernel(const __nv_bfloat16* __restrict__ kv, l
     }
 }
 
+// The same in pieces of eight entries, where every part starts on 16 bytes.
+__global__ void __launch_bounds__(256) pack_latent_heads_vec_kernel(const uint4* __restrict__ kv, long long ldkv8, const uint4* __restrict__ row,
+                                                                    int H, int D8, int Rd8, int Dv8, int C8,
+                                                                    const int* __restrict__ seq_of, const int* __restrict__ pos,
+                                                                    const int* __restrict__ table, int table_width,
+                                                                    uint4* __restrict__ K, uint4* __restrict__ V) {
+    const int t = blockIdx.x;
+    const int b = seq_of[t];
+    if (b < 0) return;
+    const int p = pos[t];
+    const int page = table[size_t(b) * table_width + (p >> GB_PAGE_SHIFT)], place = p & (GB_PAGE - 1);
+    const int hk = D8 + Rd8;
+    const uint4* kvr = kv + size_t(t) * ldkv8;
+    const uint4* rr = row + size_t(t) * (C8 + Rd8) + C8;
+    for (int idx = threadIdx.x; idx < H * hk; idx += blockDim.x) {
+        const int h = idx / hk, d = idx - h * hk;
+        K[((size_t(page) * H + h) * GB_PAGE + place) * hk + d] = d < D8 ? kvr[h * D8 + d] : rr[d - D8];
+    }
+    for (int idx = threadIdx.x; idx < H * Dv8; idx += blockDim.x) {
+        const int h = idx / Dv8, d = idx - h * Dv8;
+        V[((size_t(page) * H + h) * GB_PAGE + place) * Dv8 + d] = kvr[size_t(H) * D8 + idx];
+    }
+}
+
 GB_API int gb_pack_latent_heads(const void* kv, long long ldkv, const void* row, int T, int H, int D, int Rd, int Dv, int C,
                                 const int* seq_of, const int* pos, const int* table, int table_width, void* K, void* V,
                                 cudaStream_t stream) {
     GB_REQUIRE(H > 0 && D > 0 && Rd >= 0 && Dv > 0 && C > 0 && table_width > 0, "gb_pack_latent_heads: bad sizes");
     if (T == 0) return 0;
+    if (D % 8 == 0 && Rd % 8 == 0 && Dv % 8 == 0 && C % 8 == 0 && ldkv % 8 == 0 && gb_aligned(kv, 16) && gb_aligned(row, 16) &&
+        gb_aligned(K, 16) && gb_aligned(V, 16)) {
+        pack_latent_heads_vec_kernel<<<T, 256, 0, stream>>>((const uint4*)kv, ldkv / 8, (const uint4*)row, H, D / 8, Rd / 8, Dv / 8, C / 8,
+                                                            seq_of, pos, table, table_width, (uint4*)K, (uint4*)V);
+        GB_LAUNCH_OK("gb_pack_latent_heads");
+        return 0;
+    }
     pack_latent_heads_kernel<<<T, 256, 0, stream>>>((const __nv_bfloat16*)kv, ldkv, (const __nv_bfloat16*)row, H, D, Rd, Dv, C,
                                                     seq_of, pos, table, table_width, (__nv_bfloat16*)K, (__nv_bfloat16*)V);
     GB_LAUNCH_OK("gb_pack_latent_heads");
@@ -217,23 +256,23 @@ GB_API int gb_pack_latent_heads(const void* kv, long long ldkv, const void* row,
 // --------------------------------------------------- a product per head
 // out[t, h*os + o] = sum_i x[t, h*xs + i] * W[h, i, o] for o < O: every head has a matrix [I, O] of its own
 // (row-major, heads one after the other).  32-bit FMAs.  A block takes HM_TOKENS tokens, one head and 32
-// output columns; its four warps take a quarter of the inputs each (in ascending i) and the quarters are
-// added in warp order, so a token's result depends on neither the batch nor timing.  A gate multiplies every result by
+// output columns; its WARPS warps take an equal part of the inputs each (in ascending i) and the parts are
+// added in warp order (the number of warps follows from the inputs alone: heads of 256 inputs or more take 16), so a token's result depends on neither the batch nor timing.  A gate multiplies every result by
 // sigmoid(gate[t, h*O + o]).
 constexpr int HM_TOKENS = 8;
 
-template <typename TX, typename TW>
-__global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__ x, long long ldx, int xs,
+template <typename TX, typename TW, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) head_matmul_kernel(const TX* __restrict__ x, long long ldx, int xs,
                                                           const TW* __restrict__ W, int I, int O, void* __restrict__ out,
                                                           int out_dtype, long long ldo, int os, int T,
                                                           const void* __restrict__ gate, int gate_dtype, long long ldg) {
-    extern __shared__ float xt[];                     // [HM_TOKENS][I], then [4][HM_TOKENS][32] partial sums
+    extern __shared__ float xt[];                     // [HM_TOKENS][I], then [WARPS][HM_TOKENS][32] partial sums
     float* part = xt + HM_TOKENS * I;
     const int t0 = blockIdx.x * HM_TOKENS, h = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int o = blockIdx.z * 32 + lane;
     const int nt = min(HM_TOKENS, T - t0);
-    for (int idx = threadIdx.x; idx < HM_TOKENS * I; idx += 128) {
+    for (int idx = threadIdx.x; idx < HM_TOKENS * I; idx += WARPS * 32) {
         const int tt = idx / I, i = idx - tt * I;
         xt[idx] = tt < nt ? gb_to_float(x[size_t(t0 + tt) * ldx + size_t(h) * xs + i]) : 0.f;
     }
@@ -241,9 +280,10 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__
     float acc[HM_TOKENS];
 #pragma unroll
     for (int tt = 0; tt < HM_TOKENS; ++tt) acc[tt] = 0.f;
-    const int per = (I + 3) / 4, i0 = warp * per, i1 = min(I, i0 + per);
+    const int per = (I + WARPS - 1) / WARPS, i0 = warp * per, i1 = min(I, i0 + per);
     if (o < O) {
         const TW* wp = W + size_t(h) * I * O + o;
+#pragma unroll 8
         for (int i = i0; i < i1; ++i) {
             const float wv = gb_to_float(wp[size_t(i) * O]);
 #pragma unroll
@@ -253,11 +293,12 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const TX* __restrict__
 #pragma unroll
     for (int tt = 0; tt < HM_TOKENS; ++tt) part[(warp * HM_TOKENS + tt) * 32 + lane] = acc[tt];
     __syncthreads();
-    for (int idx = threadIdx.x; idx < HM_TOKENS * 32; idx += 128) {
+    for (int idx = threadIdx.x; idx < HM_TOKENS * 32; idx += WARPS * 32) {
         const int tt = idx >> 5, ol = idx & 31, oo = blockIdx.z * 32 + ol;
         if (tt < nt && oo < O) {
-            float v = ((part[(0 * HM_TOKENS + tt) * 32 + ol] + part[(1 * HM_TOKENS + tt) * 32 + ol]) +
-                             part[(2 * HM_TOKENS + tt) * 32 + ol]) + part[(3 * HM_TOKENS + tt) * 32 + ol];
+            float v = part[tt * 32 + ol];
+#pragma unroll
+            for (int w = 1; w < WARPS; ++w) v += part[(w * HM_TOKENS + tt) * 32 + ol];
             if (gate) v *= 1.f / (1.f + expf(-gb_load(gate, gate_dtype, size_t(t0 + tt) * ldg + size_t(h) * O + oo)));
             gb_store(out, out_dtype, size_t(t0 + tt) * ldo + size_t(h) * os + oo, v);
         }
@@ -271,13 +312,17 @@ GB_API int gb_head_matmul(const void* x, int x_dtype, long long ldx, int xs, con
     GB_REQUIRE(!gate || gb_is_dtype(gate_dtype), "gb_head_matmul: bad gate dtype");
     GB_REQUIRE(gb_is_dtype(x_dtype) && gb_is_dtype(w_dtype) && gb_is_dtype(out_dtype), "gb_head_matmul: bad dtype");
     GB_REQUIRE(H > 0 && H <= 65535 && I > 0 && O > 0 && xs >= I && os >= O, "gb_head_matmul: bad sizes heads=%d in=%d out=%d", H, I, O);
-    const size_t smem = (size_t(HM_TOKENS) * I + 4 * HM_TOKENS * 32) * sizeof(float);
+    const bool many = I >= 256 && I <= 960;
+    const size_t smem = (size_t(HM_TOKENS) * I + (many ? 16 : 4) * HM_TOKENS * 32) * sizeof(float);
     GB_REQUIRE(smem <= 48 * 1024, "gb_head_matmul: %d inputs per head exceed %d", I, (48 * 1024 / 4 - 4 * HM_TOKENS * 32) / HM_TOKENS);
     if (T == 0) return 0;
     dim3 grid((T + HM_TOKENS - 1) / HM_TOKENS, H, (O + 31) / 32);
     GB_REQUIRE(grid.z <= 65535, "gb_head_matmul: too many outputs per head (%d)", O);
 #define HM_LAUNCH(TX, TW)                                                                                             \
-    head_matmul_kernel<TX, TW><<<grid, 128, smem, stream>>>((const TX*)x, ldx, xs, (const TW*)W, I, O, out, out_dtype, ldo, os, T, gate, gate_dtype, ldg)
+    do {                                                                                                              \
+        if (many) head_matmul_kernel<TX, TW, 16><<<grid, 512, smem, stream>>>((const TX*)x, ldx, xs, (const TW*)W, I, O, out, out_dtype, ldo, os, T, gate, gate_dtype, ldg); \
+        else head_matmul_kernel<TX, TW, 4><<<grid, 128, smem, stream>>>((const TX*)x, ldx, xs, (const TW*)W, I, O, out, out_dtype, ldo, os, T, gate, gate_dtype, ldg); \
+    } while (0)
     if (x_dtype == GB_F32 && w_dtype == GB_F32) HM_LAUNCH(float, float);
     else if (x_dtype == GB_BF16 && w_dtype == GB_BF16) HM_LAUNCH(__nv_bfloat16, __nv_bfloat16);
     else if (x_dtype == GB_BF16 && w_dtype == GB_F32) HM_LAUNCH(__nv_bfloat16, float);
@@ -382,6 +427,105 @@ __global__ void __launch_bounds__(128) head_prep_kv_write_kernel(const HeadPrepP
     }
 }
 
+// The same for bfloat16 rows and caches whose heads start on 8 bytes, heads of up to 512 entries: one warp per head (eight to a
+// block, the heads of a token over gridDim.y blocks), four entries per lane and piece, the angles of the token's position
+// once per block.  v the same rows as k: the key's warp stores both.
+template <int NV>
+__global__ void __launch_bounds__(256) head_prep_vec_kernel(const HeadPrepParams a) {
+    extern __shared__ float hp_sm[];                  // cosines and sines [2][half], then a head per warp [8][D]
+    gb_grid_launch_dependents();
+    gb_grid_wait();
+    const int t = blockIdx.x;
+    const int b = a.seq_of[t];
+    if (b < 0) return;
+    const int p = a.pos[t];
+    const int H = a.H, G = a.G, D = a.D, Dv = a.Dv;
+    const int half = a.inv_freq ? a.rot_dims / 2 : 0;
+    float *cs = hp_sm, *sn = hp_sm + half;
+    if (half) {
+        for (int i = threadIdx.x; i < half; i += 256) sincosf(float(p) * a.inv_freq[i], &sn[i], &cs[i]);
+        __syncthreads();
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool same = a.v == a.k;
+    const int items = !a.k ? H : same ? H + G : H + 2 * G;
+    const int item = blockIdx.y * 8 + warp;
+    if (item >= items) return;
+    const size_t row = size_t(t) * size_t(a.ld);
+    const int* trow = a.table + size_t(b) * a.table_width;
+    if (item >= H + G) {                              // a value head
+        const int g = item - H - G;
+        const size_t o = row + size_t(g) * Dv, c = gb_kv_offset(trow, a.ring_pages, p, g, G, Dv, a.head_pages);
+        for (int i = 4 * lane; i < Dv; i += 128) {
+            float4 x = gb_load4(a.v, GB_BF16, o + i);
+            if (a.first_out) *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.first_out) + size_t(t) * a.ld_out + size_t(g) * Dv + i) = gb_pack4(x);
+            if (a.v_first) {
+                const float4 f = gb_load4(a.v_first, GB_BF16, size_t(t) * a.ld_first + size_t(g) * Dv + i);
+                const float l = a.lambda, m = 1.f - l;
+                x = make_float4(m * x.x + l * f.x, m * x.y + l * f.y, m * x.z + l * f.z, m * x.w + l * f.w);
+            }
+            *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.vcache) + c + i) = gb_pack4(x);
+        }
+        return;
+    }
+    const bool is_q = item < H;
+    const void* src = is_q ? (const void*)a.q : a.k;
+    const void* w = is_q ? a.wq : a.wk;
+    const size_t o = row + size_t(is_q ? item : item - H) * D;
+    const size_t c = is_q ? o : gb_kv_offset(trow, a.ring_pages, p, item - H, G, D, a.head_pages);
+    float4 x[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = 4 * lane + 128 * k;
+        x[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < D) {
+            x[k] = gb_load4(src, GB_BF16, o + i);
+            if (same && !is_q) *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.vcache) + c + i) = gb_pack4(x[k]);
+        }
+        ss = fmaf(x[k].x, x[k].x, ss); ss = fmaf(x[k].y, x[k].y, ss); ss = fmaf(x[k].z, x[k].z, ss); ss = fmaf(x[k].w, x[k].w, ss);
+    }
+    const float f = w ? 1.f / sqrtf(gb_warp_sum(ss) / float(D) + a.eps) : 1.f;
+    const float temp = is_q && a.temp_coef != 0.f ? 1.f + a.temp_coef * logf(float((p + 1) / a.temp_every) + 1.f) : 1.f;
+    float* buf = hp_sm + 2 * half + warp * D;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = 4 * lane + 128 * k;
+        if (i < D) {
+            if (w) {
+                const float4 g = gb_load4(w, a.w_dtype, i);
+                x[k] = make_float4(x[k].x * f * g.x, x[k].y * f * g.y, x[k].z * f * g.z, x[k].w * f * g.w);
+            }
+            x[k] = make_float4(x[k].x * temp, x[k].y * temp, x[k].z * temp, x[k].w * temp);
+            if (half) *reinterpret_cast<float4*>(buf + i) = x[k];
+        }
+    }
+    if (half) {
+        __syncwarp();
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            float* xe = reinterpret_cast<float*>(&x[k]);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int d = 4 * lane + 128 * k + e;
+                if (d >= 2 * half) continue;
+                const int pair = a.pairing ? d >> 1 : d < half ? d : d - half;
+                const bool first = a.pairing ? (d & 1) == 0 : d < half;
+                const float other = buf[a.pairing ? d ^ 1 : first ? d + half : d - half];
+                float y0, y1;
+                gb_rotate(first ? xe[e] : other, first ? other : xe[e], cs[pair], sn[pair], y0, y1);
+                xe[e] = first ? y0 : y1;
+            }
+        }
+    }
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(is_q ? a.q : a.kcache);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = 4 * lane + 128 * k;
+        if (i < D) *reinterpret_cast<uint2*>(dst + c + i) = gb_pack4(x[k]);
+    }
+}
+
 // q [T, H*D] (treated in place), k [T, G*D], v [T, G*Dv]: column slices of one row-major buffer, rows `ld` apart.
 // kcache [pages, G, PAGE, D], vcache [pages, G, PAGE, Dv].  v_first, first_out: [T, G*Dv] with rows of their own.
 GB_API int gb_head_prep_kv_write(void* q, const void* k, const void* v, int dtype, long long ld, int T, int H, int G, int D,
@@ -404,6 +548,23 @@ GB_API int gb_head_prep_kv_write(void* q, const void* k, const void* v, int dtyp
     a.ld_first = ld_first; a.lambda = lambda; a.first_out = first_out; a.ld_out = ld_out; a.temp_coef = temp_coef; a.temp_every = temp_every > 0 ? temp_every : 1; a.seq_of = seq_of; a.pos = pos;
     a.table = table; a.table_width = table_width; a.ring_pages = ring_pages; a.head_pages = head_pages; a.kcache = kcache;
     a.vcache = vcache; a.cache_dtype = cache_dtype;
+    const bool vec = dtype == GB_BF16 && (!k || cache_dtype == GB_BF16) && D % 4 == 0 && Dv % 4 == 0 && D <= 512 && ld % 4 == 0 &&
+                     gb_aligned(q, 8) && gb_aligned(k, 8) && gb_aligned(v, 8) && gb_aligned(kcache, 8) && gb_aligned(vcache, 8) &&
+                     (!wq || (gb_aligned(wq, w_dtype == GB_F32 ? 16 : 8) && gb_aligned(wk, w_dtype == GB_F32 ? 16 : 8))) &&
+                     (!v_first || (gb_aligned(v_first, 8) && ld_first % 4 == 0)) && (!first_out || (gb_aligned(first_out, 8) && ld_out % 4 == 0)) &&
+                     !(k && v == k && (Dv != D || v_first || first_out));
+    if (vec) {
+        const int half = inv_freq ? rot_dims / 2 : 0, items = !k ? H : v == k ? H + G : H + 2 * G;
+        const size_t smem = half ? (size_t(2) * half + size_t(8) * D) * sizeof(float) : 0;
+        if (half % 2 == 0) {                          // the heads' rows behind the angles start on 16 bytes
+            const dim3 grid(T, (items + 7) / 8);
+            if (D <= 128) gb_launch(head_prep_vec_kernel<1>, grid, dim3(256), smem, stream, a);
+            else if (D <= 256) gb_launch(head_prep_vec_kernel<2>, grid, dim3(256), smem, stream, a);
+            else gb_launch(head_prep_vec_kernel<4>, grid, dim3(256), smem, stream, a);
+            GB_LAUNCH_OK("gb_head_prep_kv_write");
+            return 0;
+        }
+    }
     head_prep_kv_write_kernel<<<T, 128, size_t(4) * D * sizeof(float), stream>>>(a);
     GB_LAUNCH_OK("gb_head_prep_kv_write");
     return 0;

@@ -81,6 +81,23 @@ __device__ __forceinline__ void gb_store(void* p, int dtype, size_t i, float v) 
     else reinterpret_cast<__nv_bfloat16*>(p)[i] = __float2bfloat16_rn(v);
 }
 
+// Four entries at once from a place that starts on four entries' bytes, as 32-bit floats; and back to bfloat16.
+__device__ __forceinline__ float4 gb_load4(const void* p, int dtype, size_t i) {
+    if (dtype == GB_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
+    const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p) + i);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ uint2 gb_pack4(const float4& v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<const unsigned*>(&a);
+    r.y = *reinterpret_cast<const unsigned*>(&b);
+    return r;
+}
+static inline bool gb_aligned(const void* p, size_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+
 // Entry of a sequence's page table that holds position `pos`: the sequence's first head_pages pages are kept
 // for ever (entries 0 .. head_pages - 1), the pages after them go round a ring of ring_pages entries behind
 // those.  head_pages 0: the ring alone.

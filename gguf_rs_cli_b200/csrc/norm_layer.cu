@@ -36,31 +36,20 @@ __device__ __forceinline__ float ln_block_sum(float v, float* red) {
     return tot;
 }
 
-__device__ __forceinline__ float4 ln_load4(const void* p, int dtype, size_t i) {
-    if (dtype == GB_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
-    const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p) + i);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ uint2 ln_pack4(const float4& v) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    uint2 r;
-    r.x = *reinterpret_cast<const unsigned*>(&a);
-    r.y = *reinterpret_cast<const unsigned*>(&b);
-    return r;
-}
-
 // NV pieces of four entries per thread: piece k of thread i starts at entry 4 * (i + k * blockDim.x)
 template <int NV>
-__global__ void __launch_bounds__(1024) layernorm_vec_kernel(const LnParams p) {
+__global__ void __launch_bounds__(NV < 4 ? 1024 : 512) layernorm_vec_kernel(const LnParams p) {
     __shared__ float red1[32], red2[32];
     const int E = p.E;
-    float4 v[NV], wv[NV];
+    float4 v[NV];
+    constexpr bool EARLY = NV <= 2;        // the weights do not depend on the kernel before this one; with many pieces their
+    float4 wv[EARLY ? NV : 1];             // registers would cost resident blocks
+    if (EARLY) {
 #pragma unroll
-    for (int k = 0; k < NV; ++k) {                             // the weights do not depend on the kernel before this one
-        const int i = 4 * (threadIdx.x + k * blockDim.x);
-        wv[k] = i < E ? ln_load4(p.w, p.w_dtype, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < (EARLY ? NV : 1); ++k) {
+            const int i = 4 * (threadIdx.x + k * blockDim.x);
+            wv[k] = i < E ? gb_load4(p.w, p.w_dtype, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
     }
     gb_grid_launch_dependents();
     gb_grid_wait();
@@ -74,15 +63,12 @@ __global__ void __launch_bounds__(1024) layernorm_vec_kernel(const LnParams p) {
             v[k] = *reinterpret_cast<const float4*>(p.x + size_t(t) * E + i);
             v[k].x *= p.alpha; v[k].y *= p.alpha; v[k].z *= p.alpha; v[k].w *= p.alpha;
             if (p.y) {
-                const float4 y = ln_load4(p.y, p.y_dtype, size_t(t) * p.ldy + i);
+                const float4 y = gb_load4(p.y, p.y_dtype, size_t(t) * p.ldy + i);
                 v[k].x += y.x; v[k].y += y.y; v[k].z += y.z; v[k].w += y.w;
             }
         }
     }
     if (p.z) {
-        float4 a[NV];
-#pragma unroll
-        for (int k = 0; k < NV; ++k) a[k] = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int r = 0; r < p.top; ++r) {
             const int pair = t * p.top + r;
             const float wr = p.weights[pair];
@@ -92,13 +78,11 @@ __global__ void __launch_bounds__(1024) layernorm_vec_kernel(const LnParams p) {
                 const int i = 4 * (threadIdx.x + k * blockDim.x);
                 if (i < E) {
                     const float4 y = *reinterpret_cast<const float4*>(zr + i);
-                    a[k].x = fmaf(wr, y.x, a[k].x); a[k].y = fmaf(wr, y.y, a[k].y);
-                    a[k].z = fmaf(wr, y.z, a[k].z); a[k].w = fmaf(wr, y.w, a[k].w);
+                    v[k].x = fmaf(wr, y.x, v[k].x); v[k].y = fmaf(wr, y.y, v[k].y);
+                    v[k].z = fmaf(wr, y.z, v[k].z); v[k].w = fmaf(wr, y.w, v[k].w);
                 }
             }
         }
-#pragma unroll
-        for (int k = 0; k < NV; ++k) { v[k].x += a[k].x; v[k].y += a[k].y; v[k].z += a[k].z; v[k].w += a[k].w; }
     }
 #pragma unroll
     for (int k = 0; k < NV; ++k) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
@@ -118,13 +102,14 @@ __global__ void __launch_bounds__(1024) layernorm_vec_kernel(const LnParams p) {
     for (int k = 0; k < NV; ++k) {
         const int i = 4 * (threadIdx.x + k * blockDim.x);
         if (i < E) {
-            const float4 o = make_float4(v[k].x * f * wv[k].x, v[k].y * f * wv[k].y, v[k].z * f * wv[k].z, v[k].w * f * wv[k].w);
+            const float4 g = EARLY ? wv[EARLY ? k : 0] : gb_load4(p.w, p.w_dtype, i);
+            const float4 o = make_float4(v[k].x * f * g.x, v[k].y * f * g.y, v[k].z * f * g.z, v[k].w * f * g.w);
             if (p.write_x) *reinterpret_cast<float4*>(p.x + size_t(t) * E + i) = o;
-            if (p.xb) *reinterpret_cast<uint2*>(p.xb + size_t(t) * E + i) = ln_pack4(o);
+            if (p.xb) *reinterpret_cast<uint2*>(p.xb + size_t(t) * E + i) = gb_pack4(o);
             if (p.h) {
                 const size_t at = size_t(blockIdx.x) * E + i;
                 if (p.h_dtype == GB_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.h) + at) = o;
-                else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.h) + at) = ln_pack4(o);
+                else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.h) + at) = gb_pack4(o);
             }
         }
     }
@@ -141,12 +126,10 @@ __global__ void __launch_bounds__(256) layernorm_kernel(const LnParams p) {
         float v = p.alpha * p.x[size_t(t) * E + i];
         if (p.y) v += gb_load(p.y, p.y_dtype, size_t(t) * p.ldy + i);
         if (p.z) {
-            float a = 0.f;
             for (int r = 0; r < p.top; ++r) {
                 const int pair = t * p.top + r;
-                a = fmaf(p.weights[pair], p.z[size_t(p.place_of ? p.place_of[pair] : pair) * E + i], a);
+                v = fmaf(p.weights[pair], p.z[size_t(p.place_of ? p.place_of[pair] : pair) * E + i], v);
             }
-            v += a;
         }
         ln_row[i] = v;
         s += v;
@@ -167,8 +150,6 @@ __global__ void __launch_bounds__(256) layernorm_kernel(const LnParams p) {
     }
 }
 
-bool ln_aligned(const void* p, int mask) { return (reinterpret_cast<uintptr_t>(p) & mask) == 0; }
-
 }  // namespace
 
 // x float32 [T, E] contiguous; y [T, E] rows ldy apart or null; z float32 [T * top, E] contiguous with weights [T, top] and
@@ -187,17 +168,19 @@ GB_API int gb_layernorm(float* x, const void* y, int y_dtype, long long ldy, con
     p.x = x; p.y = y; p.z = z; p.weights = weights; p.place_of = place_of; p.rows = rows; p.w = w; p.h = h;
     p.xb = (__nv_bfloat16*)xb; p.ldy = ldy; p.alpha = alpha; p.eps = eps; p.y_dtype = y_dtype; p.w_dtype = w_dtype;
     p.h_dtype = h_dtype; p.top = top; p.E = E; p.write_x = write_x;
-    const bool vec = E % 4 == 0 && E <= 16384 && ln_aligned(x, 15) && ln_aligned(w, w_dtype == GB_F32 ? 15 : 7) &&
-                     (!y || (ldy % 4 == 0 && ln_aligned(y, y_dtype == GB_F32 ? 15 : 7))) && (!z || ln_aligned(z, 15)) &&
-                     (!h || ln_aligned(h, h_dtype == GB_F32 ? 15 : 7)) && (!xb || ln_aligned(xb, 7));
+    const bool vec = E % 4 == 0 && E <= 16384 && gb_aligned(x, 16) && gb_aligned(w, w_dtype == GB_F32 ? 16 : 8) &&
+                     (!y || (ldy % 4 == 0 && gb_aligned(y, y_dtype == GB_F32 ? 16 : 8))) && (!z || gb_aligned(z, 16)) &&
+                     (!h || gb_aligned(h, h_dtype == GB_F32 ? 16 : 8)) && (!xb || gb_aligned(xb, 8));
     if (vec) {
         const int pieces = E / 4;
-        // one piece per thread up to 512 threads, then two, then four
-        const int nv = pieces <= 512 ? 1 : pieces <= 2048 ? 2 : 4;
+        // few rows: few pieces per thread, which shortens a row's way through the block; many rows: four pieces per thread,
+        // so that all rows of a step are under way at once (2,048 rows of 2,048: 22 us with one piece)
+        const int nv = pieces > 2048 ? 8 : n_rows >= 256 || pieces > 1024 ? 4 : pieces > 512 ? 2 : 1;
         const int threads = ((pieces + nv - 1) / nv + 31) / 32 * 32;
         if (nv == 1) gb_launch(layernorm_vec_kernel<1>, dim3(n_rows), dim3(threads), 0, stream, p);
         else if (nv == 2) gb_launch(layernorm_vec_kernel<2>, dim3(n_rows), dim3(threads), 0, stream, p);
-        else gb_launch(layernorm_vec_kernel<4>, dim3(n_rows), dim3(threads), 0, stream, p);
+        else if (nv == 4) gb_launch(layernorm_vec_kernel<4>, dim3(n_rows), dim3(threads), 0, stream, p);
+        else gb_launch(layernorm_vec_kernel<8>, dim3(n_rows), dim3(threads), 0, stream, p);
     } else {
         const size_t smem = size_t(E) * 4;
         if (smem > 48 * 1024 &&
@@ -221,7 +204,7 @@ __global__ void __launch_bounds__(128) rms_rows_kernel(const void* __restrict__ 
     float ss = 0.f;
     if (vec) {
         for (int i = 4 * lane; i < C; i += 128) {
-            const float4 v = ln_load4(in, in_dtype, size_t(t) * ldi + i);
+            const float4 v = gb_load4(in, in_dtype, size_t(t) * ldi + i);
             ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
         }
     } else {
@@ -233,10 +216,10 @@ __global__ void __launch_bounds__(128) rms_rows_kernel(const void* __restrict__ 
     const float f = 1.f / sqrtf(gb_warp_sum(ss) / float(C) + eps);
     if (vec) {
         for (int i = 4 * lane; i < C; i += 128) {
-            const float4 v = ln_load4(in, in_dtype, size_t(t) * ldi + i), g = ln_load4(w, w_dtype, i);
+            const float4 v = gb_load4(in, in_dtype, size_t(t) * ldi + i), g = gb_load4(w, w_dtype, i);
             const float4 o = make_float4(v.x * f * g.x, v.y * f * g.y, v.z * f * g.z, v.w * f * g.w);
             if (out_dtype == GB_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + size_t(t) * ldo + i) = o;
-            else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + size_t(t) * ldo + i) = ln_pack4(o);
+            else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + size_t(t) * ldo + i) = gb_pack4(o);
         }
     } else {
         for (int i = lane; i < C; i += 32)
@@ -249,8 +232,8 @@ GB_API int gb_rms_rows(const void* in, int in_dtype, long long ldi, int T, int C
     GB_REQUIRE(gb_is_dtype(in_dtype) && gb_is_dtype(w_dtype) && gb_is_dtype(out_dtype), "gb_rms_rows: bad dtype");
     GB_REQUIRE(in && w && out && T >= 0 && C > 0 && eps > 0.f && ldi >= C && ldo >= C, "gb_rms_rows: bad sizes T=%d C=%d", T, C);
     if (T == 0) return 0;
-    const bool vec = C % 4 == 0 && ldi % 4 == 0 && ldo % 4 == 0 && ln_aligned(in, in_dtype == GB_F32 ? 15 : 7) &&
-                     ln_aligned(w, w_dtype == GB_F32 ? 15 : 7) && ln_aligned(out, out_dtype == GB_F32 ? 15 : 7);
+    const bool vec = C % 4 == 0 && ldi % 4 == 0 && ldo % 4 == 0 && gb_aligned(in, in_dtype == GB_F32 ? 16 : 8) &&
+                     gb_aligned(w, w_dtype == GB_F32 ? 16 : 8) && gb_aligned(out, out_dtype == GB_F32 ? 16 : 8);
     gb_launch(rms_rows_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, in, in_dtype, ldi, T, C, w, w_dtype, eps, out, out_dtype, ldo, int(vec));
     GB_LAUNCH_OK("gb_rms_rows");
     return 0;
