@@ -91,7 +91,7 @@ def all_chosen(cfg):
     return cfg
 
 
-def make_weights(cfg, seed=0, gain=1.3):
+def make_weights(cfg, seed=0, gain=1.0):
     """name -> float32 tensor holding bfloat16 values.  Projections N(0, gain^2/in), so that rows stay of order one."""
     g = torch.Generator().manual_seed(seed)
     E, V, w = cfg["width"], cfg["vocab"], {}

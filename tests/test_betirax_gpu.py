@@ -25,9 +25,8 @@ NAMES = ["small", "wide"]
 
 def assert_close(got, want, dtype, what="", tol=None):
     """32-bit: the largest error against the largest value of the compared block.  bfloat16, row by row: the root mean
-    square of a row's error is held to 5% of the block's root mean square for a mechanism alone; of a whole model's rows
-    (peaked softmaxes pass a rounding on enlarged, from layer to layer) one in twenty may be off by more than 10%, and none
-    by more than 25%: a key left out, a wrong edge or a lost row moves results by far more, and the 32-bit runs tell."""
+    square of a row's error is held to 5% of the block's root mean square for a mechanism alone, to 10% for whole models
+    (peaked softmaxes pass a rounding on enlarged, from layer to layer; the 32-bit runs are the sharper test of those)."""
     got, want = got.detach().float().cpu(), want.detach().float().cpu()
     assert got.shape == want.shape, f"{what}: shape {tuple(got.shape)} != {tuple(want.shape)}"
     assert torch.isfinite(got).all(), f"{what}: non-finite values"
@@ -37,9 +36,8 @@ def assert_close(got, want, dtype, what="", tol=None):
         return
     g2, w2 = got.reshape(-1, got.shape[-1]), want.reshape(-1, want.shape[-1])
     rms_ref = max(float(w2.pow(2).mean().sqrt()), 1e-6)
-    rows = (g2 - w2).pow(2).mean(-1).sqrt() / rms_ref
-    worst, over = float(rows.max()), int((rows > (0.05 if tol is None else 0.1)).sum())
-    assert over <= (0 if tol is None else g2.shape[0] // 20) and worst <= 0.25, f"{what}: {over} of {g2.shape[0]} rows are off, the worst by {worst:.3f} of {rms_ref:.3e} (max error {err:.3e}, {dtype})"
+    worst, limit = float((g2 - w2).pow(2).mean(-1).sqrt().max()) / rms_ref, 0.05 if tol is None else 0.1
+    assert worst <= limit, f"{what}: a row is off by {worst:.3f} of {rms_ref:.3e} (max error {err:.3e}, {dtype})"
 
 
 def assert_model(got, want, dtype, what=""):
