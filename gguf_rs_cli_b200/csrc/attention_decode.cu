@@ -43,9 +43,11 @@ struct AdParams {
     const float* sink_values;    // ... or of the score sink_values[head] (not scaled); null: 0
     int chunk;                   // > 0: in a window's place, a token sees the earlier tokens of its own chunk of that many positions
     const float* slopes;         // [nh] or null: a score loses slopes[head] * (its distance), after the scale
+    float softcap, out_scale;    // > 0: a scaled score s becomes softcap tanh(s / softcap); a factor of every result
 };
 
 __device__ __forceinline__ float ad_gated(const AdParams& p, int t, int h, int d, float o) {
+    o *= p.out_scale;
     if (!p.gate) return o;
     const size_t at = p.gate_per_head ? size_t(h) : size_t(h) * p.hd + d;
     return o / (1.f + expf(-__bfloat162float(p.gate[size_t(t) * p.ldg + at])));
@@ -89,10 +91,11 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(AdParams p
     __shared__ float m_s[AD_WARPS][GT], l_s[AD_WARPS][GT];
     __shared__ int last_flag;
 
+    const float q_scale = p.softcap > 0.f ? p.scale_log2 / (p.softcap * 1.4426950408889634f) : p.scale_log2;
     for (int i = threadIdx.x; i < GT * HC * 64; i += AD_THREADS) {
         int gi = i / (HC * 64), d = i - gi * (HC * 64);
         float v = 0.f;
-        if (gi < heads && d < hd) v = __bfloat162float(p.q[size_t(t) * p.ldq + size_t(h0 + gi) * hd + d]) * p.scale_log2;
+        if (gi < heads && d < hd) v = __bfloat162float(p.q[size_t(t) * p.ldq + size_t(h0 + gi) * hd + d]) * q_scale;
         qs[gi][d] = v;
     }
     __syncthreads();
@@ -150,6 +153,7 @@ __global__ void __launch_bounds__(AD_THREADS) attention_decode_kernel(AdParams p
 #pragma unroll
         for (int gi = 0; gi < GT; ++gi) {
             float sc = s[gi] + __shfl_xor_sync(0xffffffffu, s[gi], 1);
+            if (p.softcap > 0.f) sc = p.softcap * 1.4426950408889634f * tanhf(sc);        // the queries came in units of the cap
             if (p.slopes) sc -= slope2[gi] * float(pos - j);
             sc = valid ? sc : -INFINITY;
             float mx = sc;
@@ -291,7 +295,7 @@ static int attention_decode_launch(const void* q, long long ldq, void* out, long
                                    const void* kcache, const void* vcache, int window, float scale, int splits,
                                    float* scratch, int* counters, int n_counters, int head_pages, int keep_first,
                                    const void* gate, long long ldg, int gate_per_head, int sink, const float* sink_values, int chunk,
-                                   const float* slopes, cudaStream_t stream) {
+                                   const float* slopes, float softcap, float out_scale, cudaStream_t stream) {
     GB_REQUIRE(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "gb_attention_decode: chunks go with neither a window nor kept positions");
     GB_REQUIRE(gb_attention_decode_supported(hd, GB_BF16, GB_BF16), "gb_attention_decode: head_dim %d must be a multiple of 16 up to 256", hd);
     GB_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0, "gb_attention_decode: %d heads are not a multiple of %d KV heads", nh, nkv);
@@ -311,6 +315,7 @@ static int attention_decode_launch(const void* q, long long ldq, void* out, long
     p.ring_pages = ring_pages; p.window = window; p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f;
     p.head_pages = head_pages; p.keep_first = keep_first; p.gate = (const __nv_bfloat16*)gate; p.ldg = ldg;
     p.gate_per_head = gate_per_head; p.sink = sink; p.sink_values = sink_values; p.chunk = chunk; p.slopes = slopes;
+    p.softcap = softcap; p.out_scale = out_scale;
     dim3 grid(T, nkv * gtiles, splits);
     int hc = (hd + 63) / 64;
     switch (gt) {
@@ -328,21 +333,22 @@ GB_API int gb_attention_decode(const void* q, long long ldq, void* out, long lon
                                const void* kcache, const void* vcache, int window, float scale, int splits,
                                float* scratch, int* counters, int n_counters, cudaStream_t stream) {
     return attention_decode_launch(q, ldq, out, ldo, T, nh, nkv, hd, seq_of, pos, table, table_width, ring_pages, kcache, vcache,
-                                   window, scale, splits, scratch, counters, n_counters, 0, 0, nullptr, 0, 0, 0, nullptr, 0, nullptr, stream);
+                                   window, scale, splits, scratch, counters, n_counters, 0, 0, nullptr, 0, 0, 0, nullptr, 0, nullptr, 0.f, 1.f, stream);
 }
 
 // The same behind a window that keeps the sequence's first keep_first positions visible (their pages are the first
 // head_pages entries of the page table), the result multiplied by sigmoid(gate) when a gate [T, nh*hd] (gate_per_head:
 // [T, nh]) is given; sink: one more key without a value in the softmax's denominator, of score 0 or sink_values[head];
 // chunk: in a window's place, chunks of that many positions counted from the sequence's start; slopes [nh]: a distance bias
-// (a score loses slopes[head] times its distance).
+// (a score loses slopes[head] times its distance); softcap c > 0: a scaled score s becomes c tanh(s / c), before the bias;
+// out_scale: a factor of every result.
 GB_API int gb_attention_decode_kept(const void* q, long long ldq, void* out, long long ldo, int T, int nh, int nkv, int hd,
                                     const int* seq_of, const int* pos, const int* table, int table_width, int ring_pages,
                                     const void* kcache, const void* vcache, int window, float scale, int splits,
                                     float* scratch, int* counters, int n_counters, int head_pages, int keep_first,
                                     const void* gate, long long ldg, int gate_per_head, int sink, const float* sink_values,
-                                    int chunk, const float* slopes, cudaStream_t stream) {
+                                    int chunk, const float* slopes, float softcap, float out_scale, cudaStream_t stream) {
     return attention_decode_launch(q, ldq, out, ldo, T, nh, nkv, hd, seq_of, pos, table, table_width, ring_pages, kcache, vcache,
                                    window, scale, splits, scratch, counters, n_counters, head_pages, keep_first, gate, ldg,
-                                   gate_per_head, sink, sink_values, chunk, slopes, stream);
+                                   gate_per_head, sink, sink_values, chunk, slopes, softcap, out_scale, stream);
 }

@@ -13,7 +13,7 @@
 // multiplied by sigmoid(gate) entry by entry, or by one number per head; the softmax's denominator may count one
 // more key that has no value (a sink), of score 0 or of a learned score per head (not scaled).  Instead of a window
 // the keys may come in chunks of `chunk` positions counted from the sequence's start: a token sees the earlier tokens of
-// its own chunk only.  A distance bias takes slopes[head] * (i - j) off the scaled score of query i and key j.
+// its own chunk only.  A softcap c turns every scaled score s into c tanh(s / c).  A distance bias takes slopes[head] * (i - j) off the scaled score of query i and key j.
 #include <math.h>
 
 #include "common.cuh"
@@ -32,7 +32,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
     const int* __restrict__ table, int table_width, int ring_pages, const TC* __restrict__ kc,
     const TC* __restrict__ vc, int window, float scale, int head_pages, int keep_first, const void* __restrict__ gate,
     int gate_dtype, long long ldg, int gate_per_head, int sink, const float* __restrict__ sink_values, int chunk,
-    const float* __restrict__ slopes) {
+    const float* __restrict__ slopes, float softcap, float out_scale) {
     int t = blockIdx.x, h = blockIdx.y;
     int b = seq_of[t];
     size_t orow = size_t(t) * ldo + size_t(h) * hdv;
@@ -120,6 +120,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
             for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], gb_to_float(kr[d]), dot);
             s = dot * scale;
         }
+        if (softcap > 0.f && valid) s = softcap * tanhf(s / softcap);
         if (slopes) s -= slope * float(p - j);               // an unseen key's score stays -infinity
         float m_new = fmaxf(m, gb_warp_max(s));
         float alpha = (m == -INFINITY) ? 0.f : expf(m - m_new);
@@ -181,7 +182,7 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
     for (int d = threadIdx.x; d < hdv; d += blockDim.x) {
         float o = 0.f;
         for (int w = 0; w < AG_WARPS; ++w) o += acc_s[w][d] * wgt[w];
-        o = o * down / L;
+        o = o * down / L * out_scale;
         if (gate) o *= 1.f / (1.f + expf(-gb_load(gate, gate_dtype, size_t(t) * ldg + (gate_per_head ? size_t(h) : size_t(h) * hdv + d))));
         gb_store(out, out_dtype, orow + d, o);
     }
@@ -190,13 +191,15 @@ __global__ void __launch_bounds__(AG_WARPS * 32) attention_generic_kernel(
 // q: [T, nh, hd] with rows ldq elements apart (already rotated); out: [T, nh*hdv] with rows ldo
 // apart.  seq_of[t] is the token's row in the page table (or -1 for padding, which gives
 // zeros), pos[t] its position.  window 0 means all earlier keys.  Keys [pages, nkv, PAGE, hd]; values
-// [pages, nkv, PAGE, v_row] of which the first hdv entries count (hdv = v_row = hd for ordinary heads).
+// [pages, nkv, PAGE, v_row] of which the first hdv entries count (hdv = v_row = hd for ordinary heads).  softcap 0: none;
+// out_scale multiplies every result.
 GB_API int gb_attention_generic(const void* q, int q_dtype, long long ldq, void* out, int out_dtype, long long ldo,
                                 int T, int nh, int nkv, int hd, int hdv, int v_row, const int* seq_of, const int* pos,
                                 const int* table, int table_width, int ring_pages, const void* kcache,
                                 const void* vcache, int cache_dtype, int window, float scale, int head_pages, int keep_first,
                                 const void* gate, int gate_dtype, long long ldg, int gate_per_head, int sink,
-                                const float* sink_values, int chunk, const float* slopes, cudaStream_t stream) {
+                                const float* sink_values, int chunk, const float* slopes, float softcap, float out_scale,
+                                cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(q_dtype) && gb_is_dtype(out_dtype) && gb_is_dtype(cache_dtype), "gb_attention_generic: bad dtype");
     GB_REQUIRE(hd > 0 && hd <= AG_MAX_HD, "gb_attention_generic: head_dim %d is not in 1..%d", hd, AG_MAX_HD);
     GB_REQUIRE(hdv > 0 && hdv <= AG_MAX_HD && v_row >= hdv, "gb_attention_generic: value size %d (rows of %d) is not in 1..%d", hdv, v_row, AG_MAX_HD);
@@ -211,7 +214,7 @@ GB_API int gb_attention_generic(const void* q, int q_dtype, long long ldq, void*
 #define AG_LAUNCH(TC, MAX_HD)                                                                                     \
     attention_generic_kernel<TC, MAX_HD><<<grid, AG_WARPS * 32, 0, stream>>>(                                     \
         q, q_dtype, ldq, out, out_dtype, ldo, nh, nkv, hd, hdv, v_row, seq_of, pos, table, table_width, ring_pages, \
-        (const TC*)kcache, (const TC*)vcache, window, scale, head_pages, window > 0 ? keep_first : 0, gate, gate_dtype, ldg, gate_per_head, sink, sink_values, chunk, slopes)
+        (const TC*)kcache, (const TC*)vcache, window, scale, head_pages, window > 0 ? keep_first : 0, gate, gate_dtype, ldg, gate_per_head, sink, sink_values, chunk, slopes, softcap, out_scale)
     const bool small = hd <= 256 && hdv <= 256, mid = hd <= AG_MID_HD && hdv <= AG_MID_HD;
     if (cache_dtype == GB_F32) {
         if (small) AG_LAUNCH(float, 256);

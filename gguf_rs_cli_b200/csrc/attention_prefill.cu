@@ -7,7 +7,7 @@
 // cores through mma.sync m16n8k16 (bf16 in, f32 accumulate): 8 warps x 16 queries;
 // K and V pages are double-buffered in shared memory with cp.async.
 //
-// Sizes: head_dim 64 or 128 here (other sizes take the generic kernel), any group
+// Sizes: head_dim 64, 96 or 128 here (other sizes take the generic kernel), any group
 // size, any window, sequences that start anywhere in their cache.  Behind a window the
 // sequence's first keep_first positions may stay visible (their pages are walked first);
 // the result may be multiplied by sigmoid(gate) entry by entry.
@@ -50,6 +50,8 @@ struct ApParams {
     const float* sink_values;        // ... or of the score sink_values[head] (not scaled); null: 0
     int chunk;                       // > 0: in a window's place, a token sees the earlier tokens of its own chunk of that many positions
     const float* slopes;             // [nh] or null: a score loses slopes[head] * (its distance), after the scale (EXACT only)
+    float softcap;                   // > 0: a scaled score s becomes softcap tanh(s / softcap) (EXACT only)
+    float out_scale;                 // multiplies every result
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -79,8 +81,10 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 }
 
 // Element offset of (row, 16-byte chunk) in a tile of HD-wide bf16 rows whose chunks are
-// XOR-swizzled within groups of 8 so that ldmatrix rows fall into distinct banks.
+// XOR-swizzled within groups of 8 (heads of 96: of 4, as rows then start half a bank line apart) so that ldmatrix rows
+// fall into distinct banks.
 template <int HD> __device__ __forceinline__ int swz(int row, int chunk) {
+    if (HD % 64) return row * HD + ((chunk ^ ((row >> 1) & 3)) << 3);
     return row * HD + (((chunk & ~7) | ((chunk ^ row) & 7)) << 3);
 }
 
@@ -150,9 +154,10 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
     const int pq0 = r0 < rows ? start + q0 + r0 : -1, pq1 = r1 < rows ? start + q0 + r1 : -1;
     const int lo0 = gb_first_visible(pq0, p.window, p.chunk), lo1 = gb_first_visible(pq1, p.window, p.chunk);
 
-    // with a distance bias the scores are brought into the exponent's units (and biased) before the softmax
-    const bool biased = EXACT && p.slopes;
-    const float slope2 = biased ? p.slopes[h] * 1.4426950408889634f : 0.f;
+    // with a softcap or a distance bias the scores are brought into the exponent's units before the softmax
+    const bool capped = EXACT && p.softcap > 0.f, biased = EXACT && (p.slopes || capped);
+    const float slope2 = EXACT && p.slopes ? p.slopes[h] * 1.4426950408889634f : 0.f;
+    const float to_cap = capped ? p.scale_log2 / (p.softcap * 1.4426950408889634f) : 0.f, cap2 = p.softcap * 1.4426950408889634f;
     const float sl2 = biased ? 1.f : p.scale_log2;
 
     float o[OT][4];
@@ -198,8 +203,10 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
         for (int j = 0; j < NT; ++j) {
             if (biased) {
                 const float d0 = float(pq0 - key0 - 8 * j), d1 = float(pq1 - key0 - 8 * j);
-                s[j][0] = s[j][0] * p.scale_log2 - slope2 * d0; s[j][1] = s[j][1] * p.scale_log2 - slope2 * (d0 - 1.f);
-                s[j][2] = s[j][2] * p.scale_log2 - slope2 * d1; s[j][3] = s[j][3] * p.scale_log2 - slope2 * (d1 - 1.f);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[j][e] = capped ? cap2 * tanhf(s[j][e] * to_cap) : s[j][e] * p.scale_log2;
+                s[j][0] -= slope2 * d0; s[j][1] -= slope2 * (d0 - 1.f);
+                s[j][2] -= slope2 * d1; s[j][3] -= slope2 * (d1 - 1.f);
             }
             if (need_mask) {
                 int ka = key0 + 8 * j, kb2 = ka + 1;
@@ -289,7 +296,7 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
         if (m0 != -INFINITY) l0 += exp2f(sv - m0 * sl2);
         if (m1 != -INFINITY) l1 += exp2f(sv - m1 * sl2);
     }
-    float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+    float inv0 = l0 > 0.f ? p.out_scale / l0 : 0.f, inv1 = l1 > 0.f ? p.out_scale / l1 : 0.f;
     const bool entry_gate = p.gate && !p.gate_per_head;
     if (p.gate && p.gate_per_head) {
         if (r0 < rows) inv0 *= 1.f / (1.f + expf(-__bfloat162float(p.gate[size_t(tok0 + r0) * p.ldg + h])));
@@ -335,7 +342,7 @@ template <int HD, bool EXACT> int launch_ap(const ApParams& p, int n_tiles, cuda
 }  // namespace
 
 GB_API int gb_attention_prefill_supported(int hd, int cache_dtype, int q_dtype) {
-    return cache_dtype == GB_BF16 && q_dtype == GB_BF16 && (hd == 64 || hd == 128);
+    return cache_dtype == GB_BF16 && q_dtype == GB_BF16 && (hd == 64 || hd == 96 || hd == 128);
 }
 
 // Queries per tile: the caller lists, for every sequence of the step, tiles (sequence row, first query)
@@ -347,13 +354,13 @@ GB_API int gb_attention_prefill(const void* q, long long ldq, void* out, long lo
                                 const int* table, int table_width, int ring_pages, const void* kcache,
                                 const void* vcache, int window, float scale, int exact, int head_pages, int keep_first,
                                 const void* gate, long long ldg, int gate_per_head, int sink, const float* sink_values, int chunk,
-                                const float* slopes, cudaStream_t stream) {
-    GB_REQUIRE(gb_attention_prefill_supported(hd, GB_BF16, GB_BF16), "gb_attention_prefill: head_dim %d is not 64 or 128", hd);
+                                const float* slopes, float softcap, float out_scale, cudaStream_t stream) {
+    GB_REQUIRE(gb_attention_prefill_supported(hd, GB_BF16, GB_BF16), "gb_attention_prefill: head_dim %d is not 64, 96 or 128", hd);
     GB_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0, "gb_attention_prefill: bad head counts %d / %d", nh, nkv);
     GB_REQUIRE(n_tiles <= 65535, "gb_attention_prefill: %d tiles of queries are too many for one launch", n_tiles);
     GB_REQUIRE(window >= 0 && ring_pages > 0 && table_width > 0 && head_pages >= 0, "gb_attention_prefill: bad cache geometry");
     GB_REQUIRE(keep_first >= 0, "gb_attention_prefill: a negative number of kept positions");
-    GB_REQUIRE(!slopes || exact, "gb_attention_prefill: a distance bias goes with 32-bit weights");
+    GB_REQUIRE(!(slopes || softcap > 0.f) || exact, "gb_attention_prefill: a distance bias or a softcap goes with 32-bit weights");
     GB_REQUIRE(!gate || gate_per_head || ((ldg % 2) == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0), "gb_attention_prefill: misaligned gate");
     GB_REQUIRE((ldq % 8) == 0 && (ldo % 2) == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0 &&
                    (reinterpret_cast<uintptr_t>(kcache) & 15) == 0 && (reinterpret_cast<uintptr_t>(vcache) & 15) == 0,
@@ -366,6 +373,7 @@ GB_API int gb_attention_prefill(const void* q, long long ldq, void* out, long lo
     p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
     p.head_pages = head_pages; p.keep_first = keep_first; p.gate = (const __nv_bfloat16*)gate; p.ldg = ldg;
     p.gate_per_head = gate_per_head; p.sink = sink; p.sink_values = sink_values; p.chunk = chunk; p.slopes = slopes;
-    if (exact) return hd == 64 ? launch_ap<64, true>(p, n_tiles, stream) : launch_ap<128, true>(p, n_tiles, stream);
-    return hd == 64 ? launch_ap<64, false>(p, n_tiles, stream) : launch_ap<128, false>(p, n_tiles, stream);
+    p.softcap = softcap; p.out_scale = out_scale;
+    if (exact) return hd == 64 ? launch_ap<64, true>(p, n_tiles, stream) : hd == 96 ? launch_ap<96, true>(p, n_tiles, stream) : launch_ap<128, true>(p, n_tiles, stream);
+    return hd == 64 ? launch_ap<64, false>(p, n_tiles, stream) : hd == 96 ? launch_ap<96, false>(p, n_tiles, stream) : launch_ap<128, false>(p, n_tiles, stream);
 }

@@ -560,37 +560,37 @@ GB_API int gb_gemm_tc_supported(const void* X, long long ldx, const void* W, lon
 static int gemm_tc_impl(const void* X, long long ldx, const void* W, long long ldw, const void* bias, int bias_dtype,
                         void* out, int out_dtype, long long ldo, int T, int N, int K, float* scratch, int* counters,
                         int n_counters, int sms, int swiglu_features, int gate_act, const float* row_ssq, int ssq_parts, int norm_size,
-                        float eps, float* resid_x, void* resid_xb, float* ssq_out, long long ld_x, cudaStream_t stream);
+                        float eps, float* resid_x, void* resid_xb, float* ssq_out, long long ld_x, float resid_scale, cudaStream_t stream);
 
 GB_API int gb_gemm_tc(const void* X, long long ldx, const void* W, long long ldw, const void* bias, int bias_dtype,
                       void* out, int out_dtype, long long ldo, int T, int N, int K, float* scratch, int* counters,
                       int n_counters, int sms, int swiglu_features, cudaStream_t stream) {
     return gemm_tc_impl(X, ldx, W, ldw, bias, bias_dtype, out, out_dtype, ldo, T, N, K, scratch, counters, n_counters, sms,
-                        swiglu_features, GB_ACT_SILU, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, 0, stream);
+                        swiglu_features, GB_ACT_SILU, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr, 0, 1.f, stream);
 }
 
 // The same product with a deferred RMS norm on its input and/or a residual epilogue:
 //  - row_ssq [ssq_parts, T] (f32): X holds rows that were not normalised (the norm's weight is folded into W);
 //    every result is scaled by 1 / sqrt(sum_i row_ssq[i][t] / norm_size + eps) before bias and activation;
-//  - resid_x [T, N] f32 with pitch ld_x: instead of writing `out`, x += result (+ bias) in place, resid_xb (bf16,
+//  - resid_x [T, N] f32 with pitch ld_x: instead of writing `out`, x += resid_scale * (result + bias) in place, resid_xb (bf16,
 //    same pitch) gets the rounded copy, and ssq_out [ceil(N/128), T] the sums of squares of the new x over each
 //    tile of 128 features: the row_ssq of the product that reads xb next.
 GB_API int gb_gemm_tc_fused(const void* X, long long ldx, const void* W, long long ldw, const void* bias, int bias_dtype,
                             void* out, int out_dtype, long long ldo, int T, int N, int K, float* scratch, int* counters,
                             int n_counters, int sms, int swiglu_features, int gate_act, const float* row_ssq, int ssq_parts,
                             int norm_size, float eps, float* resid_x, void* resid_xb, float* ssq_out, long long ld_x,
-                            cudaStream_t stream) {
+                            float resid_scale, cudaStream_t stream) {
     GB_REQUIRE(!row_ssq || (ssq_parts > 0 && norm_size > 0 && eps > 0.f), "gb_gemm_tc_fused: bad norm parameters");
     GB_REQUIRE(!resid_x || (resid_xb && ssq_out && ld_x >= N && !swiglu_features), "gb_gemm_tc_fused: bad residual parameters");
     GB_REQUIRE(!swiglu_features || gate_act == GB_ACT_SILU || gate_act == GB_ACT_GELU_TANH, "gb_gemm_tc_fused: unknown gate activation %d", gate_act);
     return gemm_tc_impl(X, ldx, W, ldw, bias, bias_dtype, out, out_dtype, ldo, T, N, K, scratch, counters, n_counters, sms,
-                        swiglu_features, gate_act, row_ssq, ssq_parts, norm_size, eps, resid_x, resid_xb, ssq_out, ld_x, stream);
+                        swiglu_features, gate_act, row_ssq, ssq_parts, norm_size, eps, resid_x, resid_xb, ssq_out, ld_x, resid_scale, stream);
 }
 
 static int gemm_tc_impl(const void* X, long long ldx, const void* W, long long ldw, const void* bias, int bias_dtype,
                         void* out, int out_dtype, long long ldo, int T, int N, int K, float* scratch, int* counters,
                         int n_counters, int sms, int swiglu_features, int gate_act, const float* row_ssq, int ssq_parts, int norm_size,
-                        float eps, float* resid_x, void* resid_xb, float* ssq_out, long long ld_x, cudaStream_t stream) {
+                        float eps, float* resid_x, void* resid_xb, float* ssq_out, long long ld_x, float resid_scale, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(out_dtype) && (!bias || gb_is_dtype(bias_dtype)), "gb_gemm_tc: bad dtype");
     GB_REQUIRE(T >= 0 && N > 0 && K > 0, "gb_gemm_tc: bad sizes T=%d N=%d K=%d", T, N, K);
     GB_REQUIRE(swiglu_features >= 0 && (resid_x || ldo >= (swiglu_features ? swiglu_features : N)), "gb_gemm_tc: output pitch %lld too small", ldo);
@@ -611,7 +611,7 @@ static int gemm_tc_impl(const void* X, long long ldx, const void* W, long long l
     p.swiglu = swiglu_features > 0 ? gate_act : 0; p.N_out = swiglu_features; p.sms = sms;
     cut.fill(p);
     p.row_ssq = row_ssq; p.ssq_parts = ssq_parts; p.norm_size = norm_size; p.eps = eps;
-    p.resid_x = resid_x; p.resid_xb = (__nv_bfloat16*)resid_xb; p.ssq_out = ssq_out; p.ld_x = ld_x;
+    p.resid_x = resid_x; p.resid_xb = (__nv_bfloat16*)resid_xb; p.ssq_out = ssq_out; p.ld_x = ld_x; p.resid_scale = resid_scale;
     CUtensorMap mw, mx;
     if (tensor_map_2d(W, N, K, ldw, BM, &mw)) return 1;
     if (bn == 256 && g_pair && cut.cut == CUT_WHOLE) {
@@ -658,7 +658,7 @@ GB_API int gb_gemm_tc_grouped(const void* X, long long ldx, const void* W, long 
     p.n_ctas = 0; p.tiles = int(tiles); p.cut = CUT_WHOLE; p.per_tile = p.extra = 0;
     p.total_its = int(tiles * kb); p.its_each = p.its_rest = 0;
     p.row_ssq = nullptr; p.ssq_parts = 0; p.norm_size = 0; p.eps = 0.f;
-    p.resid_x = nullptr; p.resid_xb = nullptr; p.ssq_out = nullptr; p.ld_x = 0;
+    p.resid_x = nullptr; p.resid_xb = nullptr; p.ssq_out = nullptr; p.ld_x = 0; p.resid_scale = 1.f;
     p.group_t = group_t;
     CUtensorMap mw, mx, mo;
     if (tensor_map_2d(W, (long long)G * N, K, ldw, BM, &mw)) return 1;
@@ -779,7 +779,7 @@ GB_API int gb_gemm_tc_noalloc(const void* X, long long ldx, const void* W, long 
     p.swiglu = 0; p.N_out = 0; p.sms = d->sms;
     cut.fill(p);
     p.row_ssq = nullptr; p.ssq_parts = 0; p.norm_size = 0; p.eps = 0.f;
-    p.resid_x = nullptr; p.resid_xb = nullptr; p.ssq_out = nullptr; p.ld_x = 0;
+    p.resid_x = nullptr; p.resid_xb = nullptr; p.ssq_out = nullptr; p.ld_x = 0; p.resid_scale = 1.f;
     CUtensorMap mw, mx;
     if (encode_map_2d(W, N, K, ldw, BM, &mw)) return 1;
     if (encode_map_2d(X, T, K, ldx, bn, &mx)) return 1;

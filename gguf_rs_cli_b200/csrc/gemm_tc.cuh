@@ -51,6 +51,7 @@ struct TcParams {
     // features of x^2 goes to ssq_out[feature tile][t] for the norm that comes next
     float* resid_x;
     __nv_bfloat16* resid_xb;
+    float resid_scale;           // x += resid_scale * result
     float* ssq_out;
     long long ld_x;
     // several products in one launch (the kernel that pairs two SMs only): X and out hold the problems' rows one after
@@ -222,7 +223,7 @@ __device__ __forceinline__ void tc_finish_chunk(const TcParams& p, int n0, int t
         for (int jj = 0; jj < 16; ++jj) v[jj] *= rstd_s[min(c0 + jj, BN - 1)];
     }
     if (p.resid_x) {
-        // x += result; the bf16 copy and the tile's share of sum(x^2) per token for the next norm.
+        // x += resid_scale * result; the bf16 copy and the tile's share of sum(x^2) per token for the next norm.
         // All of x is read before anything is written, so that the loads are in flight together.
         float xv[16];
 #pragma unroll
@@ -234,7 +235,7 @@ __device__ __forceinline__ void tc_finish_chunk(const TcParams& p, int n0, int t
             float sq = 0.f;
             if (n < p.N && mine(c0 + jj)) {
                 const size_t at = size_t(t0 + c0 + jj) * p.ld_x + n;
-                const float xn = xv[jj] + v[jj] + bias;
+                const float xn = fmaf(p.resid_scale, v[jj] + bias, xv[jj]);
                 p.resid_x[at] = xn;
                 p.resid_xb[at] = __float2bfloat16_rn(xn);
                 sq = xn * xn;

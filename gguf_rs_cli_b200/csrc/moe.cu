@@ -127,7 +127,8 @@ template <typename TW>
 __global__ void __launch_bounds__(256) moe_router_kernel(const void* __restrict__ x, int x_dtype, long long ldx, int K,
                                                          const TW* __restrict__ w, int E, int n_groups, int keep, int top,
                                                          float scale, int* __restrict__ ids, float* __restrict__ weights,
-                                                         int softmax, const float* __restrict__ corr) {
+                                                         int softmax, const float* __restrict__ corr, const float* __restrict__ zbias,
+                                                         float* __restrict__ gate) {
     extern __shared__ float moe_xs[];
     __shared__ float z[MOE_MAX_EXPERTS];
     __shared__ float s[MOE_MAX_EXPERTS];
@@ -138,9 +139,13 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const void* __restrict_
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int i = threadIdx.x; i < K; i += blockDim.x) moe_xs[i] = gb_load(x, x_dtype, size_t(t) * ldx + i);
     __syncthreads();
-    for (int e = warp; e < E; e += (blockDim.x >> 5)) {
+    const int n_rows = gate ? E + 1 : E;             // one more row of w: a gate per token
+    for (int e = warp; e < n_rows; e += (blockDim.x >> 5)) {
         const float v = gb_warp_sum(moe_row_dot<TW>(w + size_t(e) * K, moe_xs, K, lane));
-        if (lane == 0) z[e] = v;
+        if (lane == 0) {
+            if (e < E) z[e] = zbias ? v + zbias[e] : v;
+            else gate[t] = 1.f / (1.f + expf(-v));
+        }
     }
     __syncthreads();
     if (warp == 0)
@@ -256,10 +261,11 @@ __global__ void moe_pair_sum_kernel(const float* __restrict__ z, const float* __
     out[i] = accumulate ? out[i] + acc : acc;
 }
 
-// x [T, K] rows ldx apart (the rows the router reads, 32-bit where the caller has them); w [E, K] contiguous.
+// x [T, K] rows ldx apart (the rows the router reads, 32-bit where the caller has them); w [E, K] contiguous.  zbias [E] or
+// null: added to the logits.  gate [T] or null: w has a row E as well, and gate[t] = sigmoid(w_E x_t).
 GB_API int gb_moe_router(const void* x, int x_dtype, long long ldx, int T, int K, const void* w, int w_dtype, int E, int n_groups,
                          int keep, int top, float scale, int* ids, float* weights, int softmax, const float* corr,
-                         cudaStream_t stream) {
+                         const float* zbias, float* gate, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(x_dtype) && gb_is_dtype(w_dtype), "gb_moe_router: bad dtype");
     GB_REQUIRE(E > 0 && E <= MOE_MAX_EXPERTS && K > 0, "gb_moe_router: %d experts (1..%d)", E, MOE_MAX_EXPERTS);
     GB_REQUIRE(n_groups > 0 && E % n_groups == 0 && keep > 0 && keep <= n_groups, "gb_moe_router: %d experts in %d groups, %d kept", E, n_groups, keep);
@@ -268,10 +274,10 @@ GB_API int gb_moe_router(const void* x, int x_dtype, long long ldx, int T, int K
     const size_t smem = size_t(K) * 4;
     if (w_dtype == GB_F32) {
         if (moe_smem((const void*)moe_router_kernel<float>, smem + 20 * 1024, "gb_moe_router")) return 1;
-        moe_router_kernel<float><<<T, 256, smem, stream>>>(x, x_dtype, ldx, K, (const float*)w, E, n_groups, keep, top, scale, ids, weights, softmax, corr);
+        moe_router_kernel<float><<<T, 256, smem, stream>>>(x, x_dtype, ldx, K, (const float*)w, E, n_groups, keep, top, scale, ids, weights, softmax, corr, zbias, gate);
     } else {
         if (moe_smem((const void*)moe_router_kernel<__nv_bfloat16>, smem + 20 * 1024, "gb_moe_router")) return 1;
-        moe_router_kernel<__nv_bfloat16><<<T, 256, smem, stream>>>(x, x_dtype, ldx, K, (const __nv_bfloat16*)w, E, n_groups, keep, top, scale, ids, weights, softmax, corr);
+        moe_router_kernel<__nv_bfloat16><<<T, 256, smem, stream>>>(x, x_dtype, ldx, K, (const __nv_bfloat16*)w, E, n_groups, keep, top, scale, ids, weights, softmax, corr, zbias, gate);
     }
     GB_LAUNCH_OK("gb_moe_router");
     return 0;

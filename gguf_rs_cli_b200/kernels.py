@@ -80,7 +80,8 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
                       kcache: torch.Tensor, vcache: Optional[torch.Tensor], window: int, scale: float,
                       v_dim: Optional[int] = None, keep_first: int = 0, head_pages: int = 0,
                       gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                      chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      chunk: int = 0, slopes: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                      out_scale: float = 1.0) -> torch.Tensor:
     """v_dim: entries of a value when they differ from a key's head_dim.  vcache None: the values are the
     first v_dim entries of the key rows themselves (one latent row per position serves as key and value).
     keep_first: with a window, the sequence's first positions that stay visible behind it; their pages are the first
@@ -88,7 +89,8 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
     sigmoid(gate); a gate [T, heads] holds one number per head.  sink: the softmax's denominator counts one more key
     of score 0 that has no value, or of the score sink_values[head] (float32 [heads], not scaled).  chunk: instead of a
     window, a token sees the earlier tokens of its own chunk of that many positions, counted from the sequence's start.
-    slopes float32 [heads]: slopes[head] times the distance of query and key is taken off every scaled score."""
+    softcap c > 0: a scaled score s becomes c tanh(s / c).  slopes float32 [heads]: slopes[head] times the distance of query
+    and key is taken off every scaled (and capped) score.  out_scale: a factor of every result, applied in 32-bit."""
     _cuda(q, out, seq_of, pos, table, kcache, vcache, gate, sink_values)
     _check_slopes(slopes, n_heads)
     T = q.shape[0]
@@ -103,7 +105,7 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
          ptr(kcache), ptr(kcache if vcache is None else vcache), dtype_code(kcache), int(window or 0), float(scale),
          int(head_pages), int(keep_first or 0), ptr(gate), 0 if gate is None else dtype_code(gate),
          0 if gate is None else gate.stride(0), int(per_head), int(bool(sink) or sink_values is not None), ptr(sink_values),
-         int(chunk or 0), ptr(slopes), stream_ptr())
+         int(chunk or 0), ptr(slopes), float(softcap), float(out_scale), stream_ptr())
     return out
 
 
@@ -447,17 +449,23 @@ def _check_correction(correction: Optional[torch.Tensor], n: int) -> None:
 
 
 def moe_router(x: torch.Tensor, w: torch.Tensor, n_groups: int, keep: int, top: int, scale: float, ids: torch.Tensor,
-               weights: torch.Tensor, softmax: bool = False, correction: Optional[torch.Tensor] = None) -> None:
+               weights: torch.Tensor, softmax: bool = False, correction: Optional[torch.Tensor] = None,
+               bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """The router's product x w^T (32-bit sums) and the choice of moe_route in one kernel; x [T, K], w [experts, K].
+    bias float32 [experts]: added to the logits.  gate float32 [T]: w has one more row behind the experts'; gate[t] receives
+    the sigmoid of its product with x_t.
     softmax: scores are softmax over all experts instead of sigmoids; correction float32 [experts]: added to the scores
     for the choice, not for the weights."""
     _cuda(x, w, ids, weights)
     T, K = x.shape
     assert x.stride(1) == 1 and w.is_contiguous() and w.shape[1] == K and ids.dtype == torch.int32 and weights.dtype == torch.float32
     assert ids.shape == (T, top) and weights.shape == (T, top) and ids.is_contiguous() and weights.is_contiguous()
-    _check_correction(correction, w.shape[0])
-    call("gb_moe_router", ptr(x), dtype_code(x), x.stride(0), T, K, ptr(w), dtype_code(w), w.shape[0], int(n_groups), int(keep),
-         int(top), float(scale), ptr(ids), ptr(weights), int(bool(softmax)), ptr(correction), stream_ptr())
+    n = w.shape[0] - (gate is not None)
+    _check_correction(correction, n)
+    _check_correction(bias, n)
+    assert gate is None or (gate.is_cuda and gate.dtype == torch.float32 and gate.numel() == T and gate.is_contiguous())
+    call("gb_moe_router", ptr(x), dtype_code(x), x.stride(0), T, K, ptr(w), dtype_code(w), n, int(n_groups), int(keep),
+         int(top), float(scale), ptr(ids), ptr(weights), int(bool(softmax)), ptr(correction), ptr(bias), ptr(gate), stream_ptr())
 
 
 def moe_gate_up(h: torch.Tensor, ids: torch.Tensor, w_gate: torch.Tensor, w_up: torch.Tensor, limit: float,
@@ -789,6 +797,89 @@ def layernorm(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, 
          0 if h is None else dtype_code(h), ptr(xb), int(write_x), stream_ptr())
 
 
+def add_rmsnorm_terms(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out: torch.Tensor,
+                      scale: float = 1.0, y_gate: Optional[torch.Tensor] = None, routed: Optional[tuple] = None,
+                      rows: Optional[torch.Tensor] = None, write_x: bool = True) -> torch.Tensor:
+    """v = x + scale * (y_gate y + the routed rows), out = v / sqrt(mean(v^2) + eps) * weight, row by row in 32-bit; v goes
+    back to x (float32 [T, E]) with write_x.  y [T, E] or None; y_gate float32 [T]: a factor per row of y (None: 1);
+    routed = (z, weights, place_of) as layernorm takes it; rows: int32 row numbers to gather (then out has len(rows) rows)."""
+    z, wts, place = routed if routed is not None else (None, None, None)
+    _cuda(x, y, weight, y_gate, z, wts, place, rows, out)
+    T, E = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and weight.numel() == E and weight.is_contiguous()
+    assert y is None or (y.shape == (T, E) and y.stride(1) == 1)
+    assert y_gate is None or (y is not None and y_gate.dtype == torch.float32 and y_gate.numel() == T and y_gate.is_contiguous())
+    top = 0
+    if z is not None:
+        top = wts.shape[1]
+        assert z.dtype == torch.float32 and z.shape == (T * top, E) and z.is_contiguous()
+        assert wts.dtype == torch.float32 and wts.shape == (T, top) and wts.is_contiguous()
+        assert place is None or (place.dtype == torch.int32 and place.numel() == T * top and place.is_contiguous())
+    n = T if rows is None else rows.numel()
+    assert out.shape == (n, E) and out.is_contiguous() and not (write_x and rows is not None)
+    call("gb_add_rmsnorm_terms", ptr(x), ptr(y), 0 if y is None else dtype_code(y), 0 if y is None else y.stride(0), ptr(y_gate),
+         ptr(z), ptr(wts), ptr(place), top, float(scale), ptr(weight), dtype_code(weight), float(eps), ptr(rows), n, E, ptr(out),
+         dtype_code(out), int(write_x), stream_ptr())
+    return out
+
+
+def scale_rows_(x: torch.Tensor, factor: torch.Tensor) -> torch.Tensor:
+    """x[t,:] *= factor[t] in place (float32, contiguous)."""
+    _cuda(x, factor)
+    T, E = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and factor.dtype == torch.float32 and factor.numel() == T and factor.is_contiguous()
+    call("gb_scale_rows", ptr(x), ptr(factor), T, E, stream_ptr())
+    return x
+
+
+def rglru(u: torch.Tensor, y: torch.Tensor, z: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+          state: torch.Tensor, out: torch.Tensor, ctx, blocks: int) -> torch.Tensor:
+    """The real-gated linear recurrence per channel, from and into state [slots, width] (float32): with r = sigmoid(z_r +
+    bias_r), i = sigmoid(z_i + bias_i), log a = -rate r, S <- a S + sqrt(1 - a^2) i u, out = S gelu_tanh(y).  u, y, out
+    [T, width]; z float32 [T, 2 width]: for every block of width / blocks channels its r columns, then its i columns;
+    bias_r, bias_i, rate float32 [width].  Prompts of more than 128 tokens run in segments of 64 side by side (three launches)."""
+    _cuda(u, y, z, bias_r, bias_i, rate, state, out)
+    T, W = u.shape
+    assert y.shape == (T, W) and out.shape == (T, W) and u.dtype == y.dtype == out.dtype and W % blocks == 0
+    assert u.stride(1) == 1 and y.stride(1) == 1 and out.stride(1) == 1
+    assert z.dtype == torch.float32 and z.shape == (T, 2 * W) and z.stride(1) == 1
+    for t in (bias_r, bias_i, rate):
+        assert t.dtype == torch.float32 and t.numel() == W and t.is_contiguous()
+    assert state.dtype == torch.float32 and state.shape[1:] == (W,) and state.is_contiguous()
+    n = native.library().gb_rglru_segment_floats(ctx.B, int(ctx.max_qlen), W)
+    seg = ctx.ws.get("rglru.segments", (n,), torch.float32) if n else None
+    call("gb_rglru", ptr(u), ptr(y), dtype_code(u), u.stride(0), ptr(z), y.stride(0), z.stride(0), ptr(bias_r), ptr(bias_i),
+         ptr(rate), ptr(state), ptr(out), dtype_code(out), out.stride(0), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), T, ctx.B, W,
+         int(blocks), int(ctx.max_qlen), ptr(seg), stream_ptr())
+    if seg is not None:
+        native.count_launches(2)
+    return out
+
+
+def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: Optional[torch.Tensor], rotary_dim: int, pairing: int,
+              k_scale: float, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, ctx, n_heads: int, dim: int,
+              vdim: int) -> torch.Tensor:
+    """Linear attention with one fixed decay per head, from and into state [slots, heads, dim, vdim] (float32):
+    S <- decay S + k' v^T, out = S^T q', with q' the rotated query and k' the rotated key times k_scale (inv_freq None: no
+    rotation).  q, k [T, heads*dim], v [T, heads*vdim]: column slices of one buffer; decay float32 [heads]; out float32
+    [T, heads*vdim].  Two launches (five where a sequence brings more than 256 tokens)."""
+    _cuda(q, k, v, inv_freq, decay, state, out)
+    T, ld = q.shape[0], q.stride(0)
+    assert k.stride(0) == ld and v.stride(0) == ld and q.dtype == k.dtype == v.dtype
+    assert q.stride(1) == 1 and k.stride(1) == 1 and v.stride(1) == 1
+    assert q.shape == k.shape == (T, n_heads * dim) and v.shape == (T, n_heads * vdim)
+    assert decay.dtype == torch.float32 and decay.numel() == n_heads and decay.is_contiguous()
+    assert state.dtype == torch.float32 and state.shape[1:] == (n_heads, dim, vdim) and state.is_contiguous()
+    assert out.dtype == torch.float32 and out.shape == (T, n_heads * vdim) and out.stride(1) == 1
+    scratch, seg = _walk_scratch(ctx, n_heads, dim, vdim)
+    call("gb_retention", ptr(q), ptr(k), ptr(v), dtype_code(q), ld, ptr(ctx.pos), ptr(inv_freq), int(rotary_dim), int(pairing),
+         float(k_scale), ptr(decay), ptr(state), ptr(out), out.stride(0), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), T, ctx.B,
+         n_heads, dim, vdim, ptr(scratch), int(ctx.max_qlen), ptr(seg), stream_ptr())
+    if seg is not None:
+        native.count_launches(3)
+    return out
+
+
 def rms_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
     """out[t,:] = x[t,:] / sqrt(mean(x[t,:]^2) + eps) * weight (32-bit sums); x may be a block of columns."""
     _cuda(x, weight, out)
@@ -899,14 +990,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
             split_k: bool = True, swiglu_features: int = 0, row_ssq: Optional[torch.Tensor] = None, ssq_parts: int = 0,
             norm_size: int = 0, eps: float = 0.0, resid_x: Optional[torch.Tensor] = None,
             resid_xb: Optional[torch.Tensor] = None, ssq_out: Optional[torch.Tensor] = None,
-            gate_activation: str = "silu") -> Optional[torch.Tensor]:
+            gate_activation: str = "silu", resid_scale: float = 1.0) -> Optional[torch.Tensor]:
     """bf16 x bf16 -> f32 accumulate on tcgen05; out bf16 or f32.  Refuses what
     gemm_tc_supported refuses.  With swiglu_features = F, w is interleave_gate_up(gate, up)
     and out [T, F] = act(x gate^T) * (x up^T), act = gate_activation (GATE_ACTS).
 
     row_ssq [ssq_parts, T]: x holds rows whose RMS norm is deferred (its weight folded into w); each
     token's results are scaled by 1 / sqrt(sum_i row_ssq[i, t] / norm_size + eps).
-    resid_x (f32 [T, N]): instead of writing `out`, resid_x += result in place, resid_xb gets the
+    resid_x (f32 [T, N]): instead of writing `out`, resid_x += resid_scale * result in place, resid_xb gets the
     bfloat16 copy and ssq_out [ceil(N/128), T] the sums of squares per tile of 128 features."""
     _cuda(x, w, bias, out, row_ssq, resid_x, resid_xb, ssq_out)
     T, K = x.shape
@@ -931,7 +1022,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out:
          ptr(counters), 0 if counters is None else counters.numel(), sc.sms, int(swiglu_features),
          GATE_ACTS[gate_activation], ptr(row_ssq),
          int(ssq_parts), int(norm_size), float(eps), ptr(resid_x), ptr(resid_xb), ptr(ssq_out),
-         0 if resid_x is None else resid_x.stride(0), stream_ptr())
+         0 if resid_x is None else resid_x.stride(0), float(resid_scale), stream_ptr())
     return out
 
 
@@ -1025,19 +1116,21 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_head
                      splits: Optional[int] = None, mma: Optional[bool] = None, max_kv: Optional[int] = None,
                      rope: Optional[tuple] = None, keep_first: int = 0, head_pages: int = 0,
                      gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                     chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     chunk: int = 0, slopes: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                     out_scale: float = 1.0) -> torch.Tensor:
     """One token per sequence over the bf16 cache; all heads of a group share one pass over
     the keys and values.  mma: the tensor-core kernel (head sizes 64 and 128; the default
     where it fits) or the CUDA-core one (any head size that is a multiple of 16).
     rope = (k, v, inv_freq, rotary_dim, pairing), tensor-core kernel only: q, k and v are the
     unrotated projections; the kernel rotates q and k and writes k and v into the cache itself
     (k and v None: it reads another run's cache and only rotates q).
-    keep_first, head_pages, gate, sink, sink_values, chunk, slopes (CUDA-core kernel only): as attention_generic."""
+    keep_first, head_pages, gate, sink, sink_values, chunk, slopes, softcap, out_scale (CUDA-core kernel only): as
+    attention_generic."""
     _check_slopes(slopes, n_heads)
     _cuda(q, out, seq_of, pos, table, kcache, vcache, gate, sink_values)
     assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == n_heads and sink_values.is_contiguous())
     sink = bool(sink) or sink_values is not None
-    kept = bool(keep_first or head_pages or gate is not None or sink or chunk or slopes is not None)
+    kept = bool(keep_first or head_pages or gate is not None or sink or chunk or slopes is not None or softcap or out_scale != 1.0)
     assert not kept or (mma is False and rope is None)
     assert gate is None or gate.dtype == torch.bfloat16
     per_head = _gate_per_head(gate, out, n_heads)
@@ -1071,7 +1164,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_head
              ptr(seq_of), ptr(pos), ptr(table), table.shape[1], ring_pages, ptr(kcache), ptr(vcache), int(window or 0),
              float(scale), splits, ptr(scratch), ptr(counters), 0 if counters is None else counters.numel(), int(head_pages),
              int(keep_first or 0), ptr(gate), 0 if gate is None else gate.stride(0), int(per_head), int(bool(sink)),
-             ptr(sink_values), int(chunk or 0), ptr(slopes), stream_ptr())
+             ptr(sink_values), int(chunk or 0), ptr(slopes), float(softcap), float(out_scale), stream_ptr())
         return out
     call(entry, ptr(q), q.stride(0), ptr(out), out.stride(0), T, n_heads, n_kv_heads, head_dim,
          ptr(seq_of), ptr(pos), ptr(table), table.shape[1], ring_pages, ptr(kcache), ptr(vcache), int(window or 0),
@@ -1106,13 +1199,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
                       table: torch.Tensor, ring_pages: int, kcache: torch.Tensor, vcache: torch.Tensor, window: int,
                       scale: float, tc: Optional[bool] = None, exact: bool = False, keep_first: int = 0, head_pages: int = 0,
                       gate: Optional[torch.Tensor] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
-                      chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      chunk: int = 0, slopes: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                      out_scale: float = 1.0) -> torch.Tensor:
     """Many tokens per sequence over the bf16 cache (which already holds their keys and
     values), flash style.  tc: both products on tcgen05 with S and PV in TMEM (the default where it
-    fits), else on mma.sync; both take head sizes 64 and 128.  exact (mma.sync kernel only): the
+    fits), else on mma.sync; both take head sizes 64 and 128, the latter 96 too.  exact (mma.sync kernel only): the
     attention weights stay 32-bit, split into three bfloat16 terms for the product with the values.
-    keep_first, head_pages, gate, sink, sink_values, chunk, slopes (mma.sync kernel only; slopes with exact): as
-    attention_generic."""
+    keep_first, head_pages, gate, sink, sink_values, chunk, slopes, softcap, out_scale (mma.sync kernel only; slopes and
+    softcap with exact): as attention_generic."""
     _check_slopes(slopes, n_heads)
     _cuda(q, out, tiles, cu, starts, qlens, table, kcache, vcache, gate, sink_values)
     assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == n_heads and sink_values.is_contiguous())
@@ -1121,7 +1215,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
     per_head = _gate_per_head(gate, out, n_heads)
     assert q.stride(1) == 1 and out.stride(1) == 1 and out.shape == (q.shape[0], n_heads * head_dim)
     assert q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and kcache.dtype == torch.bfloat16
-    plain = not (exact or keep_first or head_pages or gate is not None or sink or chunk or slopes is not None)
+    plain = not (exact or keep_first or head_pages or gate is not None or sink or chunk or slopes is not None or softcap or out_scale != 1.0)
     if tc is None:
         tc = attention_prefill_tc_supported(q, kcache, head_dim) and plain
     assert not tc or plain
@@ -1135,7 +1229,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_hea
          tiles.numel() // 2, ptr(cu), ptr(starts), ptr(qlens), ptr(table), table.shape[1], ring_pages, ptr(kcache),
          ptr(vcache), int(window or 0), float(scale), int(bool(exact)), int(head_pages), int(keep_first or 0), ptr(gate),
          0 if gate is None else gate.stride(0), int(per_head), int(bool(sink)), ptr(sink_values), int(chunk or 0),
-         ptr(slopes), stream_ptr())
+         ptr(slopes), float(softcap), float(out_scale), stream_ptr())
     return out
 
 

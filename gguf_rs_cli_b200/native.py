@@ -135,14 +135,14 @@ _SIGNATURES = {
     "gb_embed": [_P, _I, _P, _I, _I, _I, _F, _P, _P],
     "gb_embed_shadow": [_P, _I, _P, _I, _I, _I, _F, _P, _P, _P, _P],
     "gb_gemm_tc_grouped": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _P],
-    "gb_gemm_tc_fused": [_P, _L, _P, _L, _P, _I, _P, _I, _L, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _L, _P],
+    "gb_gemm_tc_fused": [_P, _L, _P, _L, _P, _I, _P, _I, _L, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P, _P, _L, _F, _P],
     "gb_add_rmsnorm": [_P, _P, _I, _I, _L, _P, _I, _I, _P, _I, _F, _P, _I, _I, _P],
     "gb_rope_kv_write": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _P],
     "gb_swiglu": [_P, _L, _P, _I, _I, _I, _I, _P],
     "gb_zero_rows": [_P, _P, _I, _I, _P],
     "gb_gemm_generic": [_P, _I, _L, _P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _P],
     "gb_attention_generic": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _I, _F, _I, _I, _P, _I, _L, _I, _I,
-                             _P, _I, _P, _P],
+                             _P, _I, _P, _F, _F, _P],
     "gb_add_dyt": [_P, _P, _I, _I, _L, _P, _I, _I, _P, _P, _I, _F, _P, _I, _I, _P],
     "gb_scale": [_P, _L, _F, _P],
     "gb_short_conv_silu": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _L, _P],
@@ -163,7 +163,7 @@ _SIGNATURES = {
     "gb_gla": [_P, _P, _P, _I, _L, _P, _I, _L, _P, _I, _F, _F, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
     "gb_gla_segment_floats": [_I, _I, _I, _I, _I],
     "gb_gla_scratch_floats": [_I, _I, _I, _I],
-    "gb_moe_router": [_P, _I, _L, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P, _P],
+    "gb_moe_router": [_P, _I, _L, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P, _P, _P, _P],
     "gb_moe_route": [_P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _P, _P],
     "gb_moe_gate_up": [_P, _I, _L, _I, _I, _I, _I, _P, _P, _P, _I, _F, _P, _I, _I, _P],
     "gb_moe_down": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _I, _L, _P],
@@ -182,6 +182,11 @@ _SIGNATURES = {
     "gb_selective_scan_segment_floats": [_I, _I, _I, _I],
     "gb_norm_sandwich": [_P, _P, _I, _L, _P, _I, _L, _P, _P, _F, _P, _P, _I, _F, _P, _I, _P, _P, _I, _I, _P],
     "gb_layernorm": [_P, _P, _I, _L, _P, _P, _P, _I, _F, _P, _I, _F, _P, _I, _I, _P, _I, _P, _I, _P],
+    "gb_add_rmsnorm_terms": [_P, _P, _I, _L, _P, _P, _P, _P, _I, _F, _P, _I, _F, _P, _I, _I, _P, _I, _I, _P],
+    "gb_scale_rows": [_P, _P, _I, _I, _P],
+    "gb_rglru": [_P, _P, _I, _L, _P, _L, _L, _P, _P, _P, _P, _P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
+    "gb_rglru_segment_floats": [_I, _I, _I],
+    "gb_retention": [_P, _P, _P, _I, _L, _P, _P, _I, _I, _F, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
     "gb_rms_rows": [_P, _I, _L, _I, _I, _P, _I, _F, _P, _I, _L, _P],
     "gb_token_side_gate": [_P, _I, _L, _P, _I, _L, _I, _P, _I, _I, _I, _I, _P, _I, _L, _P],
     "gb_pack_latent_heads": [_P, _L, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P],
@@ -201,7 +206,7 @@ _SIGNATURES = {
     "gb_gemm_tc_supported": [_P, _L, _P, _L, _I],
     "gb_attention_decode": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _P],
     "gb_attention_decode_kept": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _I, _I, _P, _L, _I, _I,
-                                 _P, _I, _P, _P],
+                                 _P, _I, _P, _F, _F, _P],
     "gb_attention_decode_mma": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _P, _P, _I, _P],
     "gb_attention_decode_mma_rope": [_P, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I,
                                      _P, _P, _I, _P],
@@ -212,7 +217,7 @@ _SIGNATURES = {
     "gb_gemm_tc_set_stamps": [_P, _I, _I],
     "gb_attention_decode_scratch_floats": [_I, _I, _I, _I],
     "gb_attention_decode_supported": [_I, _I, _I],
-    "gb_attention_prefill": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _I, _I, _P, _I, _P, _P],
+    "gb_attention_prefill": [_P, _L, _P, _L, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _I, _I, _P, _I, _P, _F, _F, _P],
     "gb_attention_prefill_supported": [_I, _I, _I],
     "gb_attention_prefill_tile": [],
     "gb_attention_prefill_tc": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P, _P, _L, _I, _F, _P],
@@ -223,7 +228,7 @@ _SIGNATURES = {
     "gb_tc_status": [],
     "gb_tc_status_clear": [],
 }
-_RESTYPES = {"gb_delta_rule_scratch_floats": ctypes.c_longlong, "gb_gla_scratch_floats": ctypes.c_longlong, "gb_gla_segment_floats": ctypes.c_longlong, "gb_selective_scan_segment_floats": ctypes.c_longlong, "gb_linear_walk_scratch_floats": ctypes.c_longlong, "gb_moe_grouped_scratch_ints": ctypes.c_longlong, "gb_latent_decode_scratch_floats": ctypes.c_longlong, "gb_gemm_tc_scratch_floats": ctypes.c_longlong, "gb_attention_decode_scratch_floats": ctypes.c_longlong}
+_RESTYPES = {"gb_rglru_segment_floats": ctypes.c_longlong, "gb_delta_rule_scratch_floats": ctypes.c_longlong, "gb_gla_scratch_floats": ctypes.c_longlong, "gb_gla_segment_floats": ctypes.c_longlong, "gb_selective_scan_segment_floats": ctypes.c_longlong, "gb_linear_walk_scratch_floats": ctypes.c_longlong, "gb_moe_grouped_scratch_ints": ctypes.c_longlong, "gb_latent_decode_scratch_floats": ctypes.c_longlong, "gb_gemm_tc_scratch_floats": ctypes.c_longlong, "gb_attention_decode_scratch_floats": ctypes.c_longlong}
 
 
 def register_signature(name: str, argtypes) -> None:
@@ -259,7 +264,7 @@ def library():
 
 _launches = 0
 # kernels launched by one call of an entry point, where that is not one
-KERNELS_PER_CALL = {"gb_short_conv_silu": 2, "gb_short_conv": 2, "gb_wkv": 2, "gb_ssd": 2, "gb_delta_rule": 2, "gb_latent_decode": 2, "gb_gla": 2, "gb_moe_grouped": 4, "gb_moe_down": 2}
+KERNELS_PER_CALL = {"gb_short_conv_silu": 2, "gb_short_conv": 2, "gb_wkv": 2, "gb_ssd": 2, "gb_retention": 2, "gb_delta_rule": 2, "gb_latent_decode": 2, "gb_gla": 2, "gb_moe_grouped": 4, "gb_moe_down": 2}
 
 
 def launch_count() -> int:

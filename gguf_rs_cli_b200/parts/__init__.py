@@ -1,5 +1,5 @@
-from . import (attention, block, delta_rule, embedding, feed_forward, gla, latent_attention, norm, pair, rotary,  # noqa: F401
-               selective_scan, ssd, token_side, wkv)  # noqa: F401  (register the built-in parts)
+from . import (attention, block, delta_rule, embedding, feed_forward, gla, latent_attention, norm, pair, retention, rglru,  # noqa: F401
+               rotary, selective_scan, ssd, token_side, wkv)  # noqa: F401  (register the built-in parts)
 from .base import HostBatch, Part, RunView, StepContext, Stream, Workspace, plan_key_of
 from .linear import Linear
 from .registry import (BLOCKS, EMBEDDINGS, EXTRAS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITIONS, register_block,

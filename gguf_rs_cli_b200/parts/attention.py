@@ -38,6 +38,12 @@ And for designs without a rotation whose keys are also their values: a bias that
 keys as projected, bias included, before their norm (`values="keys"`: no v matrix, the cache holds the normed key and the
 bare one); the query temperature beside a head norm; biases on chosen projections (`bias` a sequence of names, "o" among
 them).
+
+And for designs that bound their scores: a softcap c, which turns a scaled score s into c tanh(s / c) (`softcap`); heads
+brought to unit root mean square (`qk_norm_eps`) beside any of the options above.
+
+The part may stand beside another mixer that reads the same rows (parts/pair.py): `give_projections` hands over its first and
+last product, `mix_rows` is all between them.
 """
 from __future__ import annotations
 
@@ -63,7 +69,7 @@ class Attention(Part):
     convolution on q, k and v), sink (default False; "learned": a score per head from the tensor `sink`), out_gate "head":
     one gate per head, chunk (None or C: chunks of C positions in a window's place), exact (default False), cache_span
     (when present: the positions the cache keeps, None for all, where runs with windows of their own share one cache),
-    distance_bias (default None; the exponent e), values (default None; "keys").
+    distance_bias (default None; the exponent e), values (default None; "keys"), softcap (default None).
     tensors: q [nh*hd, E], k [nkv*hd, E], v [nkv*vd, E], o [E, nh*vd], optional q_bias, k_bias, v_bias, o_bias [E];
     with head_norm_eps q_norm, k_norm [hd]; with out_gate g [nh*vd, E] ("head": [nh, E]); with v_mix the scalar v_mix;
     with conv q_conv, k_conv, v_conv [channels, taps]."""
@@ -101,6 +107,7 @@ class Attention(Part):
         if any(n not in ("q", "k", "v", "o") for n in self.biased):
             raise ValueError(f"attention: bias {bias!r} names projections that are not q, k, v, o")
         self.distance_bias = float(p.get("distance_bias") or 0.0)
+        self.softcap = float(p.get("softcap") or 0.0)
         self.keys_are_values = p.get("values") == "keys"
         if p.get("values") not in (None, "keys"):
             raise ValueError(f"attention: values {p.get('values')!r} is not None or 'keys'")
@@ -115,7 +122,9 @@ class Attention(Part):
         # heads with a norm of their own, a gate, kept first positions or mixed values: prepared by one kernel
         # (norm, rotation, mixing, cache write) and attended to with 32-bit weights
         self.prepared = bool(self.head_norm_eps is not None or self.keep_first or self.out_gate or self.v_mix or self.conv > 1
-                             or self.sink or self.chunk or self.distance_bias or self.keys_are_values or "o" in self.biased or p.get("exact"))
+                             or self.sink or self.chunk or self.distance_bias or self.keys_are_values or "o" in self.biased or self.softcap or p.get("exact"))
+        if self.head_norm_eps is not None and self.qk_norm_eps is not None:
+            raise ValueError("attention: heads have a norm with a weight (head_norm_eps) or without one (qk_norm_eps), not both")
         # where the parts of the fused projection start: q, k, v and the gate, each at a multiple of 8 rows
         self.off, rows = {}, 0
         own = 0 if self.shares_kv else 1
@@ -129,9 +138,6 @@ class Attention(Part):
         self.conv_channels = self.off["v"] + own * self.nkv * self.vd      # q, k, v and the empty rows between them
         # normalised q and k, a query temperature or values of their own size: the exact path
         self.exact = self.prepared or self.vd != self.hd or self.qk_norm_eps is not None or self.temp_coef != 0.0
-        if self.prepared and self.qk_norm_eps is not None:
-            raise ValueError("attention: qk_norm_eps goes with none of head_norm_eps, keep_first, out_gate, v_mix, conv, sink, chunk, "
-                             "distance_bias, values, a bias on o and exact")
         if self.shares_kv and self.v_mix:
             raise ValueError("attention: a layer that reads another's keys and values has no values to mix")
         if self.exact and not self.prepared and (position is not None or self.shares_kv):
@@ -229,6 +235,8 @@ class Attention(Part):
             self.q_norm, self.k_norm = store.get(req[t["q_norm"]]), store.get(req[t["k_norm"]])
             if self.q_norm.dtype != self.k_norm.dtype:
                 self.k_norm = self.k_norm.to(self.q_norm.dtype)
+        elif self.qk_norm_eps is not None:       # a norm without a weight: one whose weight is 1
+            self.q_norm = self.k_norm = torch.ones(self.hd, dtype=torch.float32, device=mats[0].device)
         self.taps = self.taps_t = None
         if self.conv > 1:
             # one convolution over all columns of q, k and v; the empty rows between them have taps of zero
@@ -255,9 +263,9 @@ class Attention(Part):
         return {"tiles": kernels.attention_prefill_tiles(batch.qlens)}
 
     def _exact_tiled(self) -> bool:
-        """Whether prompts of the exact path take the tiled kernel (bfloat16, keys and values of 64 or 128 entries
-        both) with 32-bit attention weights; other sizes and the 32-bit mode take the general kernel."""
-        return self.dtype == torch.bfloat16 and self.vd == self.hd and self.hd in (64, 128) and self._fast_masks()
+        """Whether prompts of the exact path take the tiled kernel (bfloat16, keys and values of 64, 96 or 128
+        entries both) with 32-bit attention weights; other sizes and the 32-bit mode take the general kernel."""
+        return self.dtype == torch.bfloat16 and self.vd == self.hd and self.hd in (64, 96, 128) and self._fast_masks()
 
     def _fast_masks(self) -> bool:
         """Whether the tiled and the decode kernel know this layer's mask and sink."""
@@ -293,13 +301,28 @@ class Attention(Part):
 
     V_FIRST = "attention.v_first"          # where the layer that gives its values leaves them for the step's later layers
 
+    def give_projections(self) -> Optional[Tuple[Linear, Linear]]:
+        """For a mixer that runs this one beside another: hands its first and last product over (the caller then gives `mix_rows`
+        what the first gives, and multiplies by the last itself), or None where it cannot."""
+        if not self.prepared:
+            return None
+        both, self.qkv, self.o = (self.qkv, self.o), None, None
+        return both
+
     def _forward_prepared(self, h, ctx: StepContext, run: RunView) -> torch.Tensor:
-        """One product for q, k, v and the gate; one kernel for the heads' norm, the rotation, the mixing of values and
-        the cache write; attention with 32-bit scores and weights behind the window and the kept first positions, its
-        result gated; the output projection in 32-bit results."""
-        nh, nkv, hd, vd, T = self.nh, self.nkv, self.hd, self.vd, h.shape[0]
+        """One product for q, k, v and the gate; `mix_rows`; the output projection in 32-bit results."""
         proj = self.qkv(h, ctx)
         ctx.mark("qkv")
+        out = self.mix_rows(proj, ctx, run, ctx.ws.get("attn.out", (h.shape[0], self.nh * self.vd), ctx.dtype))
+        term = self.o(out, ctx, out_dtype=torch.float32)
+        ctx.mark("o")
+        return term
+
+    def mix_rows(self, proj, ctx: StepContext, run: RunView, out, out_scale: float = 1.0) -> torch.Tensor:
+        """proj: what the first product gives; out [T, nh*vd]: the heads' results times out_scale, for the last.  One kernel for the
+        heads' norm, the rotation, the mixing of values and the cache write; attention with 32-bit scores and weights behind
+        the window and the kept first positions, its result gated."""
+        nh, nkv, hd, vd, T = self.nh, self.nkv, self.hd, self.vd, proj.shape[0]
         off = self.off
         gate = proj[:, off["g"]:off["g"] + self.gate_rows] if self.out_gate else None
         if self.conv > 1:
@@ -320,17 +343,16 @@ class Attention(Part):
             if v_first is None or v_first.shape != (T, nkv * vd):
                 raise RuntimeError("attention: no earlier layer of this step has left values of this size to mix with")
         table, pos = ctx.tables[run.group], self.position
-        kernels.head_prep_kv_write(q, k, v, nh, nkv, hd, vd, self.q_norm, self.k_norm, self.head_norm_eps or 1.0,
+        kernels.head_prep_kv_write(q, k, v, nh, nkv, hd, vd, self.q_norm, self.k_norm, self.head_norm_eps or self.qk_norm_eps or 1.0,
                                    None if pos is None else pos.inv_freq, 0 if pos is None else pos.rotary_dim,
                                    0 if pos is None else pos.pairing, v_first, self.mix, first_out, ctx.seq_of, ctx.pos, table,
                                    run.ring_pages, run.head_pages, run.k, run.v, temp_coef=self.temp_coef, temp_every=self.temp_every)
         ctx.mark("heads")
-        out = ctx.ws.get("attn.out", (T, nh * vd), ctx.dtype)
         tiles = ctx.plan_of(self).get("tiles")
         kept = dict(keep_first=self.keep_first, head_pages=run.head_pages, gate=gate, sink=self.sink, sink_values=self.sink_values,
-                    chunk=self.chunk, slopes=self.slopes)
+                    chunk=self.chunk, slopes=self.slopes, softcap=self.softcap, out_scale=out_scale)
         if not ctx.decode and tiles is not None and self._exact_tiled() and kernels.attention_prefill_supported(q, run.k, hd):
-            # prompts, keys and values of 64 or 128 entries: the tiled kernel with 32-bit weights
+            # prompts, keys and values of 64, 96 or 128 entries: the tiled kernel with 32-bit weights
             kernels.attention_prefill(q, out, nh, nkv, hd, tiles, ctx.cu, ctx.starts, ctx.qlens, table, run.ring_pages,
                                       run.k, run.v, self.window or 0, self.scale, tc=False, exact=True, **kept)
         elif ctx.decode and self._exact_decode() and kernels.attention_decode_supported(q, run.k, hd):
@@ -343,9 +365,7 @@ class Attention(Part):
             kernels.attention_generic(q, out, nh, nkv, hd, ctx.seq_of, ctx.pos, table, run.ring_pages, run.k, run.v,
                                       self.window or 0, self.scale, v_dim=vd, **kept)
         ctx.mark("attention")
-        term = self.o(out, ctx, out_dtype=torch.float32)
-        ctx.mark("o")
-        return term
+        return out
 
     def forward(self, h, ctx: StepContext, run: RunView, residual=None) -> Optional[torch.Tensor]:
         nh, nkv, hd = self.nh, self.nkv, self.hd

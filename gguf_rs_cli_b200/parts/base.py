@@ -67,11 +67,12 @@ class Workspace:
         self.device = device
         self._bufs: Dict[Tuple, torch.Tensor] = {}
 
-    def get(self, name: str, shape, dtype: torch.dtype) -> torch.Tensor:
+    def get(self, name: str, shape, dtype: torch.dtype, zeroed: bool = False) -> torch.Tensor:
+        """zeroed: the buffer holds zeros when it is made (for padding that nobody writes)."""
         key = (name, tuple(int(s) for s in shape), dtype)
         t = self._bufs.get(key)
         if t is None:
-            t = torch.empty(key[1], dtype=dtype, device=self.device)
+            t = (torch.zeros if zeroed else torch.empty)(key[1], dtype=dtype, device=self.device)
             self._bufs[key] = t
         return t
 
@@ -177,7 +178,9 @@ class Stream:
 
     def __init__(self, x: torch.Tensor):
         self.x = x
-        self.pending: Optional[torch.Tensor] = None
+        self.pending = None                   # rows, or a mixture's RoutedRows where the next norm sums them
+        self.pending_scale = 1.0              # the factor with which the pending term enters x
+        self.term_scale = 1.0                 # the factor for a part that adds its term to x itself (`residual=stream`)
         self.more: List[torch.Tensor] = []
         self.xb: Optional[torch.Tensor] = None
         self.ssq: Optional[torch.Tensor] = None
@@ -204,12 +207,13 @@ class Blend:
 
 @dataclass
 class RoutedRows:
-    """What a mixture hands over unsummed to a block whose next kernel can finish it: token t's term is base[t] (None: nothing)
+    """What a mixture hands over unsummed to a block whose next kernel can finish it: token t's term is base_gate[t] base[t] (None: nothing)
     plus sum_r weights[t, r] rows[place_of[t * top + r]] (place_of None: the pairs' own order), the choices in their order."""
     base: Optional[torch.Tensor]         # float32 [T, E]
     rows: torch.Tensor                   # float32 [T * top, E]
     weights: torch.Tensor                # float32 [T, top]
     place_of: Optional[torch.Tensor] = None
+    base_gate: Optional[torch.Tensor] = None     # float32 [T]: a factor per token of base (None: 1)
 
 
 @dataclass

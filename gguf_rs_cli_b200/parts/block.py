@@ -24,13 +24,16 @@ def own_rows(stream: Stream, ctx: StepContext):
 class PreNormBlock:
     """x += mixer(norm_m(x)); x += ff(norm_f(x)) (src/model/llama.rs:361-404).  The sums
     are not done here: each term is left pending on the stream and the next norm adds it
-    in 32-bit while it normalises."""
+    in 32-bit while it normalises.  scale: a constant factor of both terms (default 1).  unsummed: the norms behind this
+    layer take a mixture's rows unsummed (RoutedRows) and do its weighted sum in their own pass."""
 
     norm_names = ("mixer", "feed_forward")
     graph_class = ()
 
-    def __init__(self, mixer, feed_forward, norms):
+    def __init__(self, mixer, feed_forward, norms, scale: float = 1.0, unsummed: bool = False):
         self.mixer, self.feed_forward, self.norms = mixer, feed_forward, norms
+        self.scale = float(scale)
+        self.unsummed = bool(unsummed) and getattr(feed_forward, "gives_rows", False)
         self.absorbed = {"mixer": False, "feed_forward": False}
 
     def fuse(self) -> None:
@@ -45,6 +48,13 @@ class PreNormBlock:
                 self.absorbed[name] = bool(take(give()))
 
     def forward(self, stream: Stream, ctx: StepContext, run: RunView) -> None:
+        stream.term_scale = self.scale
+        try:
+            self._forward(stream, ctx, run)
+        finally:
+            stream.term_scale = 1.0
+
+    def _forward(self, stream: Stream, ctx: StepContext, run: RunView) -> None:
         h = self._norm("mixer", stream, ctx)
         ctx.mark("norm")
         if getattr(self.mixer, "accepts_residual", False):
@@ -58,6 +68,8 @@ class PreNormBlock:
         ctx.mark("ff_norm")
         if getattr(self.feed_forward, "accepts_residual", False):
             term = self.feed_forward.forward(h, ctx, residual=stream)
+        elif self.unsummed:
+            term = self.feed_forward.forward(h, ctx, unsummed=True)
         else:
             term = self.feed_forward.forward(h, ctx)
         self._add(stream, term)
@@ -67,11 +79,10 @@ class PreNormBlock:
             return self.norms[name].apply(stream, ctx, absorbed=True)
         return self.norms[name].apply(stream, ctx)
 
-    @staticmethod
-    def _add(stream: Stream, term) -> None:
+    def _add(self, stream: Stream, term) -> None:
         """A part that has added its term to the stream itself returns None."""
         if term is not None:
-            stream.pending = term
+            stream.pending, stream.pending_scale = term, self.scale
             stream.drop_shadow()
 
 

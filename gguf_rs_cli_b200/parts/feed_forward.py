@@ -120,10 +120,15 @@ class RoutedExperts(Part):
     as one product with the unit in its epilogue).  A block whose next kernel can finish the weighted sum asks for the
     experts' rows unsummed (RoutedRows).
 
+    Also: a bias on the router's logits (`router_bias=True`, tensor `router_bias`), which both the choice and the weights see,
+    and a shared expert whose result is multiplied by sigmoid(w_sg h), one number per token (`shared_gate=True`, tensor
+    `shared_gate`); its product runs with the router's.
+
     params: hidden_size, experts, top, groups, keep, scale, expert_ff, limit, shared_ff (None: no shared expert), shared_limit,
-    score ("sigmoid" or "softmax"), correction (default False), identity (default 0).  tensors: router
+    score ("sigmoid" or "softmax"), correction (default False), identity (default 0), router_bias, shared_gate (default False).  tensors: router
     [experts + identity, E]; experts: the prefix of the experts' names (<prefix><i>.gate [F, E], .up [F, E], .down [E, F]);
-    shared: the prefix of the shared expert's (.gate, .up [Fs, E], .down [E, Fs]); correction [experts + identity]."""
+    shared: the prefix of the shared expert's (.gate, .up [Fs, E], .down [E, Fs]); correction [experts + identity]; router_bias
+    [experts + identity]; shared_gate [1, E]."""
 
     def __init__(self, spec, dtype, device):
         super().__init__(spec, dtype, device)
@@ -139,6 +144,8 @@ class RoutedExperts(Part):
         if self.score not in ("sigmoid", "softmax"):
             raise ValueError(f"moe: score {self.score!r} is not one of 'sigmoid', 'softmax'")
         self.corrected = bool(p.get("correction", False))
+        self.router_bias = bool(p.get("router_bias", False))
+        self.shared_gate = bool(p.get("shared_gate", False)) and bool(self.shared_ff)
         if self.identity and self.groups != 1:
             raise ValueError("moe: identity experts go with one group of experts")
         if self.n_all % self.groups or self.keep > self.groups or self.top > self.keep * (self.n_all // self.groups):
@@ -159,11 +166,20 @@ class RoutedExperts(Part):
                     TensorRequest(t["shared"] + ".down", (E, Fs))]
         if self.corrected:
             req.append(TensorRequest(t["correction"], (self.n_all,), init="zeros"))
+        if self.router_bias:
+            req.append(TensorRequest(t["router_bias"], (self.n_all,), init="uniform:-0.1:0.1"))
+        if self.shared_gate:
+            req.append(TensorRequest(t["shared_gate"], (1, E)))
         return req
 
     def load(self, store: WeightStore) -> None:
         req = self.tensor_requests()
-        self.router = Linear(store.get(req[0]), name="moe.router")
+        by_name, t = {r.name: r for r in req}, self.spec.tensors
+        router = store.get(req[0])
+        if self.shared_gate:                     # the shared expert's gate is one more row behind the experts'
+            router = torch.cat([router, store.get(by_name[t["shared_gate"]]).to(router.dtype)], dim=0).contiguous()
+        self.router = Linear(router, name="moe.router")
+        self.logit_bias = store.get(by_name[t["router_bias"]]).to(torch.float32).contiguous() if self.router_bias else None
         mats = [store.get(r) for r in req[1:1 + 3 * self.n]]
         dt = mats[0].dtype
         # the experts' matrices side by side: [experts, F, E] twice and [experts, E, F]
@@ -171,7 +187,7 @@ class RoutedExperts(Part):
         self.w_up = torch.stack([m.to(dt) for m in mats[1::3]]).contiguous()
         self.w_down = torch.stack([m.to(dt) for m in mats[2::3]]).contiguous()
         self.shared_gate_up = self.shared_down = None
-        self.correction = store.get(req[-1]).to(torch.float32).contiguous() if self.corrected else None
+        self.correction = store.get(by_name[t["correction"]]).to(torch.float32).contiguous() if self.corrected else None
         if self.shared_ff:
             g, u, d = (store.get(r) for r in req[1 + 3 * self.n:4 + 3 * self.n])
             self.shared_tiles = None
@@ -185,6 +201,7 @@ class RoutedExperts(Part):
     BY_EXPERT = 128               # pairs per expert, on average, from which the experts run as ordinary products of their own
     BY_EXPERT_ENTRIES = 8 << 20   # ... where an expert's matrix has at least this many entries
     graph_class = ()              # grids depend on the number of tokens only
+    gives_rows = True             # forward(unsummed=True) leaves the weighted sum to the caller
     reads_stream = True           # a block that has the rows in 32-bit gives them too (x32): the router reads those
 
     def _shared(self, h, ctx: StepContext) -> torch.Tensor:
@@ -204,8 +221,10 @@ class RoutedExperts(Part):
         # the router's product in 32-bit sums, from 32-bit rows where the block has them, and its choice
         ids = ctx.ws.get("moe.ids", (T, top), torch.int32)
         weights = ctx.ws.get("moe.weights", (T, top), torch.float32)
+        gate = ctx.ws.get("moe.shared_gate", (T,), torch.float32) if self.shared_gate else None
         kernels.moe_router(h if x32 is None else x32, self.router.weight, self.groups, self.keep, top,
-                           float(self.p.get("scale", 1.0)), ids, weights, softmax=self.score == "softmax", correction=self.correction)
+                           float(self.p.get("scale", 1.0)), ids, weights, softmax=self.score == "softmax", correction=self.correction,
+                           bias=self.logit_bias, gate=gate)
         ctx.mark("router")
         out = ctx.ws.get("moe.out", (T, E), torch.float32)
         if self.shared_ff:
@@ -216,6 +235,8 @@ class RoutedExperts(Part):
         base, place_of = out if self.shared_ff else None, None
         if unsummed:
             out = None
+        elif gate is not None:
+            kernels.scale_rows_(out, gate)
         if not ctx.decode and T * top >= self.BY_EXPERT * self.n and self.F * E >= self.BY_EXPERT_ENTRIES \
                 and kernels.moe_grouped_supported(h, self.w_gate):
             # very many tokens (an expert gets 128 rows or more on average) and large experts: every expert's products on
@@ -235,4 +256,4 @@ class RoutedExperts(Part):
             got = kernels.moe_down(y, ids, weights, self.w_down, out, accumulate=bool(self.shared_ff), ws=ctx.ws,
                                    identity=self.identity, h=h)
         ctx.mark("experts")
-        return RoutedRows(base, got, weights, place_of) if unsummed else out
+        return RoutedRows(base, got, weights, place_of, gate) if unsummed else out

@@ -39,6 +39,8 @@ class RMSNorm(Part):
 
     @staticmethod
     def _terms(stream: Stream) -> list:
+        if isinstance(stream.pending, RoutedRows) or stream.pending_scale != 1.0:
+            raise RuntimeError("rmsnorm: several waiting terms, two norms at once and weights around zero go with plain rows only")
         return ([stream.pending] if stream.pending is not None else []) + list(stream.more)
 
     def apply_pair(self, stream: Stream, other: "RMSNorm", ctx: StepContext, buffers=("normed", "normed2")):
@@ -83,11 +85,21 @@ class RMSNorm(Part):
             weight = self._ones
         n = stream.x.shape[0] if rows is None else rows.numel()
         out = ctx.ws.get(buffer, (n, self.p["size"]), ctx.dtype)
-        kernels.add_rmsnorm(stream.x, stream.pending, weight, self.p["eps"], out, rows=rows, write_x=rows is None)
+        term = stream.pending
+        if isinstance(term, RoutedRows):          # a mixture's weighted sum in the same pass
+            kernels.add_rmsnorm_terms(stream.x, term.base, weight, self.p["eps"], out, scale=stream.pending_scale, y_gate=term.base_gate,
+                                      routed=(term.rows, term.weights, term.place_of), rows=rows, write_x=rows is None)
+        elif term is not None and stream.pending_scale != 1.0:
+            if term.dim() != 2:
+                raise RuntimeError("rmsnorm: a term with a factor must be one [tokens, size]")
+            kernels.add_rmsnorm_terms(stream.x, term, weight, self.p["eps"], out, scale=stream.pending_scale, rows=rows,
+                                      write_x=rows is None)
+        else:
+            kernels.add_rmsnorm(stream.x, term, weight, self.p["eps"], out, rows=rows, write_x=rows is None)
         if rows is None:
-            if stream.pending is not None:
+            if term is not None:
                 stream.drop_shadow()              # x has changed
-            stream.pending = None
+            stream.pending, stream.pending_scale = None, 1.0
         return out
 
 
@@ -143,8 +155,8 @@ class DynamicTanh(Part):
               absorbed: bool = False):
         """Adds the stream's pending term into x (32-bit) and returns tanh(alpha x) * weight + bias of all rows,
         or of `rows` only (x is then left as it is)."""
-        if stream.more:
-            raise RuntimeError("dyt: this norm adds one pending term only")
+        if stream.more or stream.pending_scale != 1.0 or isinstance(stream.pending, RoutedRows):
+            raise RuntimeError("dyt: this norm adds one pending term only, as it is")
         n = stream.x.shape[0] if rows is None else rows.numel()
         out = ctx.ws.get(buffer, (n, self.p["size"]), ctx.dtype)
         kernels.add_dyt(stream.x, stream.pending, self.weight, self.bias, self.alpha, out, rows=rows, write_x=rows is None)
@@ -176,6 +188,8 @@ class LayerNorm(Part):
         xb = ctx.ws.get("stream.xb", stream.x.shape, torch.bfloat16) if ctx.dtype == torch.bfloat16 else None
         y, routed = term, None
         if isinstance(term, RoutedRows):
+            if term.base_gate is not None:
+                kernels.scale_rows_(term.base, term.base_gate)
             y, routed = term.base, (term.rows, term.weights, term.place_of)
         kernels.layernorm(stream.x, y, self.weight, self.p["eps"], alpha=alpha, routed=routed, xb=xb)
         stream.xb, stream.ssq, stream.ssq_parts = xb, None, 0
