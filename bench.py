@@ -404,11 +404,30 @@ def betirax_config(z):
             "postln_alpha": 2.0, "layers": [layer(i) for i in range(z["layers"])]}
 
 
+def tukevik_config(z):
+    """Chunked attention (chunks of 1,024, softcap, a sink, a gate per head) beside retention (as many heads as z["heads"], all
+    entries rotated), then three recurrent blocks (gates in z["heads"] blocks, 4 taps): the mixture of mixers that the
+    design's own models have; dense feed-forwards and mixtures of 16 experts (4 of them per token, and a gated shared one:
+    Dilalix's sizes) in turn."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "shared": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 4}}
+    H = z["heads"]
+    left = {"heads": H, "kv_heads": z["kv_heads"], "dim": z["head"], "vdim": z["head"], "scale": z["head"] ** -0.5, "softcap": 30.0,
+            "mask": {"size": 1024}}
+    right = {"heads": H, "dim": z["head"], "vdim": z["head"], "decay": [1.0 - 2.0 ** (-5.0 - 5.0 * h / H) for h in range(H)],
+             "rot": {"base": 10000.0, "dims": z["head"]}}
+    pair = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.9}}
+    unit = {"type": "rglru", "mixer": {"width": z["width"], "blocks": H, "conv": 4}}
+    return {"architecture": "Tukevik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "layers": [{**(unit if i % 4 else pair), "mlp": moe if i % 2 else dense} for i in range(z["layers"])]}
+
+
 DESIGN_CONFIGS = {"debonex": debonex_config, "dilalix": dilalix_config, "nazerax": nazerax_config, "fomodra": fomodra_config,
-                  "betirax": betirax_config}
+                  "betirax": betirax_config, "tukevik": tukevik_config}
 # the closest of the other designs, which a design is measured beside
 CLOSEST = {"dilalix": [("debonex", debonex_config)], "nazerax": [("dilalix-dense", dilalix_dense_config)],
-           "fomodra": [("dilalix", dilalix_config)], "betirax": [("fomodra", fomodra_config), ("dilalix", dilalix_config)]}
+           "fomodra": [("dilalix", dilalix_config)], "betirax": [("fomodra", fomodra_config), ("dilalix", dilalix_config)],
+           "tukevik": [("dilalix", dilalix_config)]}
 
 
 def stage_times(llm, lens, starts=0, reps=3):
