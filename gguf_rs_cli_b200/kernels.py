@@ -880,6 +880,62 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: Optio
     return out
 
 
+def rotary_angles(ctx, inv_freq: torch.Tensor) -> torch.Tensor:
+    """float32 [T, pairs, 2]: cosine and sine of every token's position times every frequency, made once per step and table."""
+    key = f"rotary.angles.{inv_freq.data_ptr()}"
+    out = ctx.shared.get(key)
+    if out is None:
+        _cuda(inv_freq)
+        half = inv_freq.numel()
+        out = ctx.shared[key] = ctx.ws.get(key, (ctx.T, half, 2), torch.float32)
+        call("gb_rotary_angles", ptr(ctx.pos), ptr(inv_freq), ctx.T, half, ptr(out), stream_ptr())
+    return out
+
+
+def _retention_args(q, k, v, gate, state, out, n_heads: int, dim: int, vdim: int) -> None:
+    _cuda(q, k, v, gate, state, out)
+    T, ld = q.shape[0], q.stride(0)
+    assert k.stride(0) == ld and v.stride(0) == ld and q.dtype == k.dtype == v.dtype == gate.dtype
+    assert q.stride(1) == k.stride(1) == v.stride(1) == gate.stride(1) == out.stride(1) == 1
+    assert q.shape == k.shape == (T, n_heads * dim) and v.shape == gate.shape == out.shape == (T, n_heads * vdim)
+    assert state.dtype == torch.float32 and state.shape[1:] == (n_heads, dim, vdim) and state.is_contiguous()
+
+
+def retention_chunks_supported(q: torch.Tensor, dim: int, vdim: int) -> bool:
+    return q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and bool(native.library().gb_retention_chunks_supported(dtype_code(q), dim, vdim))
+
+
+def retention_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, inv_freq: Optional[torch.Tensor],
+                     pairing: int, k_scale: float, log2_decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, ctx, n_heads: int,
+                     dim: int, eps: float, out_scale: float = 1.0) -> torch.Tensor:
+    """retention() for steps of many tokens as matrix products over segments of 128 tokens, with the read-out's norm (no
+    weight), its SiLU gate and a factor: out [T, heads*dim] = o / sqrt(mean(o^2) + eps) * silu(gate) * out_scale, bfloat16.
+    log2_decay float32 [heads]: decays in (0, 1].  Heads that retention_chunks_supported takes.  Three launches, and one per
+    step for the angles."""
+    _retention_args(q, k, v, gate, state, out, n_heads, dim, dim)
+    assert log2_decay.dtype == torch.float32 and log2_decay.numel() == n_heads and log2_decay.is_contiguous() and out.dtype == torch.bfloat16
+    angles = None if inv_freq is None else rotary_angles(ctx, inv_freq)
+    n = native.library().gb_retention_chunk_floats(ctx.B, int(ctx.max_qlen), n_heads, dim, dim)
+    seg = ctx.ws.get("retention.segments", (n,), torch.float32)
+    call("gb_retention_chunks", ptr(q), ptr(k), ptr(v), q.stride(0), ptr(gate), gate.stride(0), ptr(angles),
+         0 if angles is None else angles.shape[1], int(pairing), float(k_scale), ptr(log2_decay), ptr(state), ptr(seg), ptr(out),
+         out.stride(0), float(eps), float(out_scale), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ctx.B, n_heads, dim,
+         int(ctx.max_qlen), stream_ptr())
+    return out
+
+
+def retention_step(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, inv_freq: Optional[torch.Tensor],
+                   rotary_dim: int, pairing: int, k_scale: float, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, ctx,
+                   n_heads: int, dim: int, vdim: int, eps: float, out_scale: float = 1.0) -> torch.Tensor:
+    """The same where every sequence brings one token, in one launch, for any sizes and dtype; decay as retention()."""
+    _retention_args(q, k, v, gate, state, out, n_heads, dim, vdim)
+    assert decay.dtype == torch.float32 and decay.numel() == n_heads and decay.is_contiguous() and ctx.max_qlen == 1
+    call("gb_retention_step", ptr(q), ptr(k), ptr(v), dtype_code(q), q.stride(0), ptr(gate), gate.stride(0), ptr(ctx.pos), ptr(inv_freq),
+         int(rotary_dim), int(pairing), float(k_scale), ptr(decay), ptr(state), ptr(out), dtype_code(out), out.stride(0), float(eps),
+         float(out_scale), ptr(ctx.cu), ptr(ctx.slots), ctx.B, n_heads, dim, vdim, stream_ptr())
+    return out
+
+
 def rms_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
     """out[t,:] = x[t,:] / sqrt(mean(x[t,:]^2) + eps) * weight (32-bit sums); x may be a block of columns."""
     _cuda(x, weight, out)

@@ -187,6 +187,11 @@ _SIGNATURES = {
     "gb_rglru": [_P, _P, _I, _L, _P, _L, _L, _P, _P, _P, _P, _P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "gb_rglru_segment_floats": [_I, _I, _I],
     "gb_retention": [_P, _P, _P, _I, _L, _P, _P, _I, _I, _F, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
+    "gb_rotary_angles": [_P, _P, _I, _I, _P, _P],
+    "gb_retention_chunks_supported": [_I, _I, _I],
+    "gb_retention_chunk_floats": [_I, _I, _I, _I, _I],
+    "gb_retention_chunks": [_P, _P, _P, _L, _P, _L, _P, _I, _I, _F, _P, _P, _P, _P, _L, _F, _F, _P, _P, _P, _I, _I, _I, _I, _P],
+    "gb_retention_step": [_P, _P, _P, _I, _L, _P, _L, _P, _P, _I, _I, _F, _P, _P, _P, _I, _L, _F, _F, _P, _P, _I, _I, _I, _I, _P],
     "gb_rms_rows": [_P, _I, _L, _I, _I, _P, _I, _F, _P, _I, _L, _P],
     "gb_token_side_gate": [_P, _I, _L, _P, _I, _L, _I, _P, _I, _I, _I, _I, _P, _I, _L, _P],
     "gb_pack_latent_heads": [_P, _L, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P],
@@ -228,7 +233,7 @@ _SIGNATURES = {
     "gb_tc_status": [],
     "gb_tc_status_clear": [],
 }
-_RESTYPES = {"gb_rglru_segment_floats": ctypes.c_longlong, "gb_delta_rule_scratch_floats": ctypes.c_longlong, "gb_gla_scratch_floats": ctypes.c_longlong, "gb_gla_segment_floats": ctypes.c_longlong, "gb_selective_scan_segment_floats": ctypes.c_longlong, "gb_linear_walk_scratch_floats": ctypes.c_longlong, "gb_moe_grouped_scratch_ints": ctypes.c_longlong, "gb_latent_decode_scratch_floats": ctypes.c_longlong, "gb_gemm_tc_scratch_floats": ctypes.c_longlong, "gb_attention_decode_scratch_floats": ctypes.c_longlong}
+_RESTYPES = {"gb_retention_chunk_floats": ctypes.c_longlong, "gb_rglru_segment_floats": ctypes.c_longlong, "gb_delta_rule_scratch_floats": ctypes.c_longlong, "gb_gla_scratch_floats": ctypes.c_longlong, "gb_gla_segment_floats": ctypes.c_longlong, "gb_selective_scan_segment_floats": ctypes.c_longlong, "gb_linear_walk_scratch_floats": ctypes.c_longlong, "gb_moe_grouped_scratch_ints": ctypes.c_longlong, "gb_latent_decode_scratch_floats": ctypes.c_longlong, "gb_gemm_tc_scratch_floats": ctypes.c_longlong, "gb_attention_decode_scratch_floats": ctypes.c_longlong}
 
 
 def register_signature(name: str, argtypes) -> None:
@@ -264,7 +269,7 @@ def library():
 
 _launches = 0
 # kernels launched by one call of an entry point, where that is not one
-KERNELS_PER_CALL = {"gb_short_conv_silu": 2, "gb_short_conv": 2, "gb_wkv": 2, "gb_ssd": 2, "gb_retention": 2, "gb_delta_rule": 2, "gb_latent_decode": 2, "gb_gla": 2, "gb_moe_grouped": 4, "gb_moe_down": 2}
+KERNELS_PER_CALL = {"gb_short_conv_silu": 2, "gb_short_conv": 2, "gb_wkv": 2, "gb_ssd": 2, "gb_retention": 2, "gb_retention_chunks": 3, "gb_delta_rule": 2, "gb_latent_decode": 2, "gb_gla": 2, "gb_moe_grouped": 4, "gb_moe_down": 2}
 
 
 def launch_count() -> int:

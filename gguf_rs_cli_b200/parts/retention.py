@@ -8,7 +8,8 @@ without a weight, multiplied by SiLU(W_g h), and projected back.  The reference 
 has attention only).
 
 q, k, v and g are one matrix after loading (each part starting at a multiple of 8 rows), so one product reads h once.
-Angles, rotated rows, decays and the state are 32-bit (csrc/retention.cu).  The part may stand beside another mixer that
+Angles, rotated rows, decays and the state are 32-bit (csrc/retention.cu: prompts in chunks on the tensor cores, single tokens in
+one pass over S, other cases by a walk over the tokens).  The part may stand beside another mixer that
 reads the same rows (parts/pair.py).
 """
 from __future__ import annotations
@@ -65,7 +66,10 @@ class Retention(Part):
             proj[at:at + w[name].shape[0]] = w[name].to(dt)
         self.proj = Linear(proj, name="retention.proj")
         self.o = Linear(w["o"], name="retention.o")
-        self.decay = torch.tensor(self.p["decay"], dtype=torch.float64).to(torch.float32).to(dev)
+        decay = torch.tensor(self.p["decay"], dtype=torch.float64)
+        self.decay = decay.to(torch.float32).to(dev)
+        # the chunked form takes powers of the decay
+        self.log2_decay = torch.log2(decay).to(torch.float32).to(dev) if bool(((decay > 0) & (decay <= 1)).all()) else None
         self._norm_weights = {}
 
     accepts_residual = True
@@ -93,13 +97,21 @@ class Retention(Part):
         """proj: what the first product gives; out [T, heads*vdim]: the gated rows times out_scale, for the last."""
         H, D, Dv, off, pos = self.H, self.D, self.Dv, self.off, self.position
         T = proj.shape[0]
+        q, k, v = proj[:, off["q"]:off["q"] + H * D], proj[:, off["k"]:off["k"] + H * D], proj[:, off["v"]:off["v"] + H * Dv]
+        gate, state, eps, k_scale = proj[:, off["g"]:off["g"] + H * Dv], ctx.state(f"run{run.index}.S"), self.p["eps"], D ** -0.5
+        inv_freq, rot, pairing = (None, 0, 0) if pos is None else (pos.inv_freq, pos.rotary_dim, pos.pairing)
+        if ctx.decode and max(D, Dv) <= 2048:
+            kernels.retention_step(q, k, v, gate, inv_freq, rot, pairing, k_scale, self.decay, state, out, ctx, H, D, Dv, eps, out_scale)
+            ctx.mark("recurrence")
+            return out
+        if self.log2_decay is not None and kernels.retention_chunks_supported(q, D, Dv):
+            kernels.retention_chunks(q, k, v, gate, inv_freq, pairing, k_scale, self.log2_decay, state, out, ctx, H, D, eps, out_scale)
+            ctx.mark("recurrence")
+            return out
         read = ctx.ws.get("retention.read", (T, H * Dv), torch.float32)
-        kernels.retention(proj[:, off["q"]:off["q"] + H * D], proj[:, off["k"]:off["k"] + H * D], proj[:, off["v"]:off["v"] + H * Dv],
-                          None if pos is None else pos.inv_freq, 0 if pos is None else pos.rotary_dim, 0 if pos is None else pos.pairing,
-                          D ** -0.5, self.decay, ctx.state(f"run{run.index}.S"), read, ctx, H, D, Dv)
+        kernels.retention(q, k, v, inv_freq, rot, pairing, k_scale, self.decay, state, read, ctx, H, D, Dv)
         ctx.mark("recurrence")
-        kernels.gated_head_norm(read, proj[:, off["g"]:off["g"] + H * Dv], self._norm_weight(out_scale, proj.device), self.p["eps"], out,
-                                H, Dv, gate_function="silu")
+        kernels.gated_head_norm(read, gate, self._norm_weight(out_scale, proj.device), eps, out, H, Dv, gate_function="silu")
         ctx.mark("head_norm")
         return out
 
