@@ -132,13 +132,46 @@ __global__ void short_conv_carry_kernel(const void* __restrict__ xin, int dtype,
     }
 }
 
+// Steps of single tokens (every sequence brings one): convolution and renewal of the carried inputs in one kernel, a thread
+// owning a channel of a sequence.  The products are added in the same order as above.
+__global__ void __launch_bounds__(128) short_conv_step_kernel(const void* __restrict__ xin, int dtype, long long ldx, int C, int K,
+                                                              const void* __restrict__ taps, int taps_dtype, float* __restrict__ state,
+                                                              const int* __restrict__ seq_of, const int* __restrict__ slots,
+                                                              void* __restrict__ out, long long ldo, const void* __restrict__ bias, int act) {
+    gb_grid_launch_dependents();
+    gb_grid_wait();
+    const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= C) return;
+    const int b = seq_of[t], slot = b < 0 ? -1 : slots[b];
+    if (slot < 0) {
+        gb_store(out, dtype, size_t(t) * ldo + c, 0.f);
+        return;
+    }
+    float* st = state + size_t(slot) * (K - 1) * C + c;
+    float x[CONV_MAX_TAPS];
+#pragma unroll
+    for (int j = 0; j < CONV_MAX_TAPS - 1; ++j) x[j] = j < K - 1 ? st[size_t(j) * C] : 0.f;
+    const float now = gb_load(xin, dtype, size_t(t) * ldx + c);
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)
+        if (j < K - 1) acc = fmaf(x[j], gb_load(taps, taps_dtype, size_t(c) * K + j), acc);
+    acc = fmaf(now, gb_load(taps, taps_dtype, size_t(c) * K + K - 1), acc);
+#pragma unroll
+    for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)
+        if (j < K - 1) st[size_t(j) * C] = j < K - 2 ? x[j + 1] : now;
+    if (bias) acc += gb_load(bias, taps_dtype, c);
+    gb_store(out, dtype, size_t(t) * ldo + c, act ? acc / (1.f + expf(-acc)) : acc);
+}
+
 // xin: [T, C] with pitch ldx (the projections' outputs); taps [C, K], last column on the current token;
 // state f32 [slots, K-1, C]; out [T, C] with pitch ldo, same dtype as xin.  The carried inputs are renewed.
 // taps_t (optional): the taps again as bfloat16 [K, C], for the kernel of 16-byte accesses.
 // bias [C] (optional, of the taps' dtype) is added to the sum; act 1: SiLU follows, 0: nothing does.
+// single: every sequence of the step brings one token (one launch instead of two).
 GB_API int gb_short_conv(const void* xin, int dtype, long long ldx, int T, int B, int C, int K, const void* taps,
                          int taps_dtype, const void* taps_t, const void* bias, int act, float* state, const int* seq_of,
-                         const int* cu, const int* slots, const int* qlens, void* out, long long ldo, cudaStream_t stream) {
+                         const int* cu, const int* slots, const int* qlens, void* out, long long ldo, int single, cudaStream_t stream) {
     GB_REQUIRE(gb_is_dtype(dtype) && gb_is_dtype(taps_dtype), "gb_short_conv: bad dtype");
     GB_REQUIRE(C > 0 && K >= 1 && K <= CONV_MAX_TAPS && ldx >= C && ldo >= C, "gb_short_conv: bad sizes C=%d taps=%d (1..%d)",
                C, K, CONV_MAX_TAPS);
@@ -147,6 +180,12 @@ GB_API int gb_short_conv(const void* xin, int dtype, long long ldx, int T, int B
     if (T == 0) return 0;
     const int threads = 128, slices = (C + threads - 1) / threads;
     GB_REQUIRE(slices <= 65535, "gb_short_conv: too many channels (%d)", C);
+    if (single && K > 1) {
+        gb_launch(short_conv_step_kernel, dim3(T, slices), dim3(threads), 0, stream, xin, dtype, ldx, C, K, taps, taps_dtype, state, seq_of,
+                  slots, out, ldo, bias, act);
+        GB_LAUNCH_OK("gb_short_conv (single tokens)");
+        return 0;
+    }
     auto aligned16 = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
     if (taps_t && dtype == GB_BF16 && C % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 && aligned16(xin) && aligned16(out) &&
         aligned16(taps_t) && (K == 1 || (reinterpret_cast<uintptr_t>(state) & 31) == 0) &&
@@ -169,9 +208,9 @@ GB_API int gb_short_conv(const void* xin, int dtype, long long ldx, int T, int B
 // The convolution followed by SiLU, without a bias.
 GB_API int gb_short_conv_silu(const void* xin, int dtype, long long ldx, int T, int B, int C, int K, const void* taps,
                               int taps_dtype, const void* taps_t, float* state, const int* seq_of, const int* cu,
-                              const int* slots, const int* qlens, void* out, long long ldo, cudaStream_t stream) {
+                              const int* slots, const int* qlens, void* out, long long ldo, int single, cudaStream_t stream) {
     return gb_short_conv(xin, dtype, ldx, T, B, C, K, taps, taps_dtype, taps_t, nullptr, 1, state, seq_of, cu, slots, qlens, out,
-                         ldo, stream);
+                         ldo, single, stream);
 }
 
 // ------------------------------------------------------------ the recurrence

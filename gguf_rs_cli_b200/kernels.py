@@ -178,7 +178,10 @@ def short_conv_silu(xin: torch.Tensor, taps: torch.Tensor, state: Optional[torch
     assert out.shape == (T, C) and out.dtype == xin.dtype
     assert state is None or (state.dtype == torch.float32 and state.shape[1:] == (K - 1, C) and state.is_contiguous())
     call("gb_short_conv_silu", ptr(xin), dtype_code(xin), xin.stride(0), T, ctx.B, C, K, ptr(taps), dtype_code(taps),
-         ptr(taps_t), ptr(state), ptr(ctx.seq_of), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ptr(out), out.stride(0), stream_ptr())
+         ptr(taps_t), ptr(state), ptr(ctx.seq_of), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ptr(out), out.stride(0),
+         int(ctx.max_qlen == 1), stream_ptr())
+    if ctx.max_qlen == 1 or K == 1:
+        native.count_launches(-1)
     return out
 
 
@@ -196,7 +199,9 @@ def short_conv(xin: torch.Tensor, taps: torch.Tensor, state: Optional[torch.Tens
     assert state is None or (state.dtype == torch.float32 and state.shape[1:] == (K - 1, C) and state.is_contiguous())
     call("gb_short_conv", ptr(xin), dtype_code(xin), xin.stride(0), T, ctx.B, C, K, ptr(taps), dtype_code(taps), ptr(taps_t),
          ptr(bias), 1 if activation else 0, ptr(state), ptr(ctx.seq_of), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ptr(out),
-         out.stride(0), stream_ptr())
+         out.stride(0), int(ctx.max_qlen == 1), stream_ptr())
+    if ctx.max_qlen == 1 or K == 1:
+        native.count_launches(-1)
     return out
 
 
@@ -837,7 +842,7 @@ def rglru(u: torch.Tensor, y: torch.Tensor, z: torch.Tensor, bias_r: torch.Tenso
     """The real-gated linear recurrence per channel, from and into state [slots, width] (float32): with r = sigmoid(z_r +
     bias_r), i = sigmoid(z_i + bias_i), log a = -rate r, S <- a S + sqrt(1 - a^2) i u, out = S gelu_tanh(y).  u, y, out
     [T, width]; z float32 [T, 2 width]: for every block of width / blocks channels its r columns, then its i columns;
-    bias_r, bias_i, rate float32 [width].  Prompts of more than 128 tokens run in segments of 64 side by side (three launches)."""
+    bias_r, bias_i, rate float32 [width].  Prompts of more than 64 tokens run in segments of 64 side by side (three launches)."""
     _cuda(u, y, z, bias_r, bias_i, rate, state, out)
     T, W = u.shape
     assert y.shape == (T, W) and out.shape == (T, W) and u.dtype == y.dtype == out.dtype and W % blocks == 0
@@ -853,6 +858,51 @@ def rglru(u: torch.Tensor, y: torch.Tensor, z: torch.Tensor, bias_r: torch.Tenso
          int(blocks), int(ctx.max_qlen), ptr(seg), stream_ptr())
     if seg is not None:
         native.count_launches(2)
+    return out
+
+
+def _rglru_args(u, y, bias_r, bias_i, rate, state, out, blocks: int) -> None:
+    _cuda(u, y, bias_r, bias_i, rate, state, out)
+    T, W = u.shape
+    assert y.shape == out.shape == (T, W) and u.dtype == y.dtype == out.dtype and W % blocks == 0
+    assert u.stride(1) == y.stride(1) == out.stride(1) == 1
+    for t in (bias_r, bias_i, rate):
+        assert t.dtype == torch.float32 and t.numel() == W and t.is_contiguous()
+    assert state.dtype == torch.float32 and state.shape[1:] == (W,) and state.is_contiguous()
+
+
+def rglru_fused_supported(u: torch.Tensor, n: int) -> bool:
+    return u.stride(0) % 8 == 0 and u.data_ptr() % 16 == 0 and bool(native.library().gb_rglru_fused_supported(dtype_code(u), n))
+
+
+def rglru_fused(u: torch.Tensor, y: torch.Tensor, gates: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+                state: torch.Tensor, out: torch.Tensor, ctx, blocks: int) -> torch.Tensor:
+    """rglru() with the gates' products in its own kernels (bfloat16, tensor cores): gates [blocks, 2n, n], a block's r rows in
+    front of its i rows.  One launch where no sequence brings more than 64 tokens, else three."""
+    _rglru_args(u, y, bias_r, bias_i, rate, state, out, blocks)
+    W = u.shape[1]
+    n = W // blocks
+    assert gates.shape == (blocks, 2 * n, n) and gates.dtype == u.dtype and gates.is_contiguous()
+    need = native.library().gb_rglru_segment_floats(ctx.B, int(ctx.max_qlen), W)
+    seg = ctx.ws.get("rglru.segments", (need,), torch.float32) if need else None
+    call("gb_rglru_fused", ptr(u), u.stride(0), ptr(y), y.stride(0), ptr(gates), ptr(bias_r), ptr(bias_i), ptr(rate), ptr(state), ptr(out),
+         out.stride(0), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ctx.B, W, int(blocks), int(ctx.max_qlen), ptr(seg), stream_ptr())
+    if seg is not None:
+        native.count_launches(2)
+    return out
+
+
+def rglru_step(u: torch.Tensor, y: torch.Tensor, gates_in: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+               state: torch.Tensor, out: torch.Tensor, ctx, blocks: int) -> torch.Tensor:
+    """The same where every sequence brings one token, in one launch, for either dtype: gates_in [blocks, n (in), 2n (out)],
+    a block's r columns in front of its i columns; blocks of up to 1,024 channels."""
+    _rglru_args(u, y, bias_r, bias_i, rate, state, out, blocks)
+    T, W = u.shape
+    n = W // blocks
+    assert gates_in.shape == (blocks, n, 2 * n) and gates_in.is_contiguous() and ctx.max_qlen == 1
+    call("gb_rglru_step", ptr(u), ptr(y), dtype_code(u), u.stride(0), y.stride(0), ptr(gates_in), dtype_code(gates_in), ptr(bias_r),
+         ptr(bias_i), ptr(rate), ptr(state), ptr(out), dtype_code(out), out.stride(0), ptr(ctx.seq_of), ptr(ctx.slots), T, W, int(blocks),
+         stream_ptr())
     return out
 
 

@@ -145,11 +145,11 @@ _SIGNATURES = {
                              _P, _I, _P, _F, _F, _P],
     "gb_add_dyt": [_P, _P, _I, _I, _L, _P, _I, _I, _P, _P, _I, _F, _P, _I, _I, _P],
     "gb_scale": [_P, _L, _F, _P],
-    "gb_short_conv_silu": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _L, _P],
+    "gb_short_conv_silu": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _L, _I, _P],
     "gb_delta_rule": [_P, _P, _P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P],
     "gb_delta_rule_scratch_floats": [_I, _I, _I, _I, _I],
     "gb_gated_head_norm": [_P, _L, _P, _I, _L, _P, _I, _F, _P, _I, _L, _I, _I, _I, _I, _I, _I, _P],
-    "gb_short_conv": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P, _L, _P],
+    "gb_short_conv": [_P, _I, _L, _I, _I, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P, _L, _I, _P],
     "gb_softcap": [_P, _L, _F, _P],
     "gb_token_shift_mix": [_P, _I, _L, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, _L, _P],
     "gb_wkv": [_P, _L, _P, _L, _P, _L, _I, _P, _I, _L, _P, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _P, _I, _P, _P],
@@ -185,6 +185,9 @@ _SIGNATURES = {
     "gb_add_rmsnorm_terms": [_P, _P, _I, _L, _P, _P, _P, _P, _I, _F, _P, _I, _F, _P, _I, _I, _P, _I, _I, _P],
     "gb_scale_rows": [_P, _P, _I, _I, _P],
     "gb_rglru": [_P, _P, _I, _L, _P, _L, _L, _P, _P, _P, _P, _P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
+    "gb_rglru_fused_supported": [_I, _I],
+    "gb_rglru_fused": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    "gb_rglru_step": [_P, _P, _I, _L, _L, _P, _I, _P, _P, _P, _P, _P, _I, _L, _P, _P, _I, _I, _I, _P],
     "gb_rglru_segment_floats": [_I, _I, _I],
     "gb_retention": [_P, _P, _P, _I, _L, _P, _P, _I, _I, _F, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
     "gb_rotary_angles": [_P, _P, _I, _I, _P, _P],

@@ -9,7 +9,8 @@ and gives W_o (S y).  The convolution's last taps - 1 inputs are per-sequence st
 mixer (src/model/llama.rs has attention only).
 
 y and x are one product.  The gates' products keep 32-bit results; gates, decays with their logarithms and exponentials
-and the state are 32-bit (csrc/rglru.cu).
+and the state are 32-bit (csrc/rglru.cu).  The gates' products are part of the recurrence's kernels, for prompts in bfloat16
+on the tensor cores and for single tokens on the CUDA cores; other cases make them first.
 """
 from __future__ import annotations
 
@@ -97,7 +98,7 @@ class GatedLinearRecurrence(Part):
         """The gates' products [T, 2 width], 32-bit results: block by block its r columns, then its i columns."""
         T, n = u.shape[0], self.n
         z = ctx.ws.get("rglru.gates", (T, 2 * self.W), torch.float32)
-        if self.gates_in is not None and (T <= 64 or ctx.dtype == torch.float32 or n % 8):
+        if self.gates_in is not None:
             return kernels.head_matmul(u, n, self.gates_in, z, 2 * n)
         for b in range(self.blocks):
             kernels.gemm(u[:, b * n:(b + 1) * n], self.gates[b], None, z[:, 2 * b * n:2 * (b + 1) * n])
@@ -111,10 +112,14 @@ class GatedLinearRecurrence(Part):
         carried = ctx.state(f"run{run.index}.conv") if self.K > 1 else None
         kernels.short_conv(proj[:, self.off_x:self.off_x + W], self.taps, carried, ctx, u, taps_t=self.taps_t, bias=self.conv_bias)
         ctx.mark("conv")
-        z = self._gates(u, ctx)
-        ctx.mark("gates")
         rows = ctx.ws.get("rglru.rows", (T, W), ctx.dtype)
-        kernels.rglru(u, proj[:, :W], z, self.r_bias, self.i_bias, self.rate, ctx.state(f"run{run.index}.S"), rows, ctx, self.blocks)
+        y, S, rates = proj[:, :W], ctx.state(f"run{run.index}.S"), (self.r_bias, self.i_bias, self.rate)
+        if ctx.decode and self.gates_in is not None:
+            kernels.rglru_step(u, y, self.gates_in, *rates, S, rows, ctx, self.blocks)
+        elif kernels.rglru_fused_supported(u, self.n):
+            kernels.rglru_fused(u, y, self.gates, *rates, S, rows, ctx, self.blocks)
+        else:
+            kernels.rglru(u, y, self._gates(u, ctx), *rates, S, rows, ctx, self.blocks)
         ctx.mark("recurrence")
         term = self.o(rows, ctx, residual=residual, out_dtype=torch.float32)
         ctx.mark("o")
