@@ -2,13 +2,15 @@
 //   r = sigmoid(z_r + b_r);  i = sigmoid(z_i + b_i);  log a = -rate_c r  (rate = 8 softplus(lam), the caller's)
 //   S <- a S + sqrt(1 - a^2) i u;   out = S gelu_tanh(y)
 // S is one 32-bit number per channel and sequence, carried from step to step; gates, decays with their logarithms and
-// exponentials and the state are 32-bit.  1 - a^2 is taken as -expm1(2 log a), which keeps its digits where a is near 1.
+// exponentials and the state are 32-bit.  Where a is near 1 its rounding to 32 bits would be the same error at every token
+// of a long memory; so a enters as a - 1 = expm1(log a): S <- S + ((a - 1) S + input), 1 - a^2 = -(a - 1)(2 + (a - 1)), and
+// products of decays are exponentials of sums of log a.
 //
 // One thread per channel walks a sequence's tokens.  Long prompts: the sequence is cut into segments that run side by
-// side.  A first pass walks every segment from zero and keeps what it ends with and the product of its decays, by which
-// a stretch of tokens multiplies the state; the state in front of each segment follows by a short walk over the segments;
-// the second pass then walks every segment from its true state and writes the results.  Prompts in bfloat16 and single
-// tokens have kernels of their own that make the gates' products as well.
+// side.  A first pass walks every segment from zero and keeps what it ends with and the sum of its log a; since a
+// stretch of tokens multiplies the state by exp(sum of log a), the state in front of each segment follows by a short walk
+// over the segments; the second pass then walks every segment from its true state and writes the results.  Prompts in
+// bfloat16 and single tokens have kernels of their own that make the gates' products as well.
 #include <math.h>
 
 #include "common.cuh"
@@ -26,15 +28,17 @@ struct RgParams {
     const float *b_r, *b_i, *rate;
     float* state;                 // [slots, W]
     void* out;
-    float* seg;                   // [B, segments, 2, W]: end state, then product of the decays; after the carry: state in front
+    float* seg;                   // [B, segments, 2, W]: end state, then sum of log a; after the carry: state in front
     long long ldu, ldy, ldz, ldo;
     const int *cu, *slots, *qlens;
     int dtype, out_dtype, W, n, mode, max_segments;
 };
 
 __device__ __forceinline__ float rg_sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
+// sqrt(1 - a^2) times v, from a - 1
+__device__ __forceinline__ float rg_input(float am1, float v) { return sqrtf(-am1 * (2.f + am1)) * v; }
 
-// mode 0: whole sequences; 1: segments from zero, keeping end state and product of the decays; 2: segments from their true state
+// mode 0: whole sequences; 1: segments from zero, keeping end state and sum of log a; 2: segments from their true state
 __global__ void __launch_bounds__(RG_THREADS) rglru_scan_kernel(const RgParams p) {
     gb_grid_launch_dependents();
     gb_grid_wait();
@@ -52,7 +56,7 @@ __global__ void __launch_bounds__(RG_THREADS) rglru_scan_kernel(const RgParams p
     }
     const int zr = (c / p.n) * 2 * p.n + c % p.n, zi = zr + p.n;
     const float br = p.b_r[c], bi = p.b_i[c], rate = p.rate[c];
-    float S = p.mode == 0 ? p.state[size_t(slot) * p.W + c] : p.mode == 2 ? rec[0] : 0.f, prod = 1.f;
+    float S = p.mode == 0 ? p.state[size_t(slot) * p.W + c] : p.mode == 2 ? rec[0] : 0.f, total = 0.f;
     for (int t0 = 0; t0 < n_tok; t0 += RG_AHEAD) {
         float zrv[RG_AHEAD], ziv[RG_AHEAD], uv[RG_AHEAD], yv[RG_AHEAD];
 #pragma unroll
@@ -70,14 +74,14 @@ __global__ void __launch_bounds__(RG_THREADS) rglru_scan_kernel(const RgParams p
         for (int j = 0; j < RG_AHEAD; ++j) {
             if (t0 + j >= n_tok) break;
             const float log_a = -rate * rg_sigmoid(zrv[j] + br);
-            const float a = expf(log_a);
-            S = fmaf(a, S, sqrtf(-expm1f(2.f * log_a)) * (rg_sigmoid(ziv[j] + bi) * uv[j]));
-            if (p.mode == 1) prod *= a;
+            const float am1 = expm1f(log_a);
+            S += fmaf(am1, S, rg_input(am1, rg_sigmoid(ziv[j] + bi) * uv[j]));
+            if (p.mode == 1) total += log_a;
             else gb_store(p.out, p.out_dtype, size_t(first + t0 + j) * p.ldo + c, S * gb_gate_act(yv[j], GB_ACT_GELU_TANH));
         }
     }
     if (p.mode == 0) p.state[size_t(slot) * p.W + c] = S;
-    else if (p.mode == 1) { rec[0] = S; rec[p.W] = prod; }
+    else if (p.mode == 1) { rec[0] = S; rec[p.W] = total; }
 }
 
 // From the segments' own end states to the states in front of them, in place, and the sequence's new state.
@@ -93,9 +97,9 @@ __global__ void __launch_bounds__(RG_THREADS) rglru_carry_kernel(float* __restri
     const int segs = (n + RG_SEGMENT - 1) / RG_SEGMENT;
     for (int s = 0; s < segs; ++s) {
         float* rec = seg + (size_t(b) * max_segments + s) * 2 * W + c;
-        const float local = rec[0], a = rec[W];
+        const float local = rec[0], am1 = expm1f(rec[W]);
         rec[0] = S;
-        S = fmaf(a, S, local);
+        S += fmaf(am1, S, local);
     }
     state[size_t(slot) * W + c] = S;
 }
@@ -103,19 +107,24 @@ __global__ void __launch_bounds__(RG_THREADS) rglru_carry_kernel(float* __restri
 // ------------------------------------------------------------------------------------------------ prompts, gates and walk in one
 // A block takes a segment of 64 tokens and 64 channels of one of the gates' blocks: the gates' products on mma.sync (the
 // segment's rows of u against the r rows and the i rows of its channels; a thread then holds both of a channel's gates for
-// its tokens), decays and inputs from the 32-bit sums, and the walk over the segment, one thread per channel.  mode as in
-// rglru_scan_kernel: the products are made twice rather than written out and read back.
+// its tokens), decays and inputs from the 32-bit sums, and the walk over the segment, one thread per channel.  Sequences of
+// one segment are finished there (mode 0).  Else (mode 1) the walk starts from zero and leaves, for every token and channel,
+// its state and what a state in front of the segment is multiplied by until there; with the states in front of the segments
+// (rglru_carry_kernel) rglru_finish_kernel then adds up and applies the other branch, entry by entry.
 constexpr int RF_TOK = RG_SEGMENT, RF_CH = 64, RF_K = 64, RF_THREADS = 256;
 
 struct RfParams {
     const __nv_bfloat16 *u, *y, *gates;      // gates [blocks, 2n, n]: a block's r rows, then its i rows
     const float *b_r, *b_i, *rate;
     float *state, *seg;
+    float* local;                            // [T, 2, W]: states of walks from zero, factors of the states in front
     __nv_bfloat16* out;
     long long ldu, ldy, ldo;
     const int *cu, *slots, *qlens;
     int W, n, slices, mode, max_segments;
 };
+
+__device__ __forceinline__ float rf_sigmoid(float v) { return __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * v)); }
 
 __device__ __forceinline__ void rf_cp16(void* dst, const void* src, bool valid) {
     const unsigned d = unsigned(__cvta_generic_to_shared(dst));
@@ -128,8 +137,9 @@ __global__ void __launch_bounds__(RF_THREADS) rglru_fused_kernel(const RfParams 
     extern __shared__ __align__(128) unsigned char rf_smem[];
     constexpr int STAGE = (RF_TOK + 2 * RF_CH) * RF_K;      // entries of one stage: u [64][64], then r and i rows [128][64]
     __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(rf_smem);
-    float* as = reinterpret_cast<float*>(rf_smem);          // [64][64] decays (then states), over the stages
+    float* as = reinterpret_cast<float*>(rf_smem);          // [64][64] a - 1 (then states), over the stages
     float* bs = as + RF_TOK * RF_CH;                        // [64][64] inputs
+    float* ls = bs + RF_TOK * RF_CH;                        // [64][64] log a, then their running sums
     gb_grid_launch_dependents();
     gb_grid_wait();
     const int blk = blockIdx.x / p.slices, c0 = (blockIdx.x % p.slices) * RF_CH;       // the gates' block, first channel in it
@@ -190,41 +200,71 @@ __global__ void __launch_bounds__(RF_THREADS) rglru_fused_kernel(const RfParams 
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int tl = tw * 16 + (lane >> 2) + (e >> 1) * 8, ch = cl + (e & 1);
-            float av = 1.f, bv = 0.f;
+            float av = 0.f, bv = 0.f, lv = 0.f;
             if (tl < n_tok && ch < nch) {
                 const int c = blk * n + c0 + ch;
-                const float log_a = -p.rate[c] * rg_sigmoid(acc[j][e] + p.b_r[c]);
-                av = expf(log_a);
-                bv = sqrtf(-expm1f(2.f * log_a)) * (rg_sigmoid(acc[j + 4][e] + p.b_i[c]) * __bfloat162float(ublk[size_t(tl) * p.ldu + c0 + ch]));
+                lv = -p.rate[c] * rf_sigmoid(acc[j][e] + p.b_r[c]);
+                av = expm1f(lv);
+                bv = rg_input(av, rf_sigmoid(acc[j + 4][e] + p.b_i[c]) * __bfloat162float(ublk[size_t(tl) * p.ldu + c0 + ch]));
             }
             as[tl * RF_CH + ch] = av;
             bs[tl * RF_CH + ch] = bv;
+            ls[tl * RF_CH + ch] = lv;
         }
     }
     __syncthreads();
     if (tid < nch) {
         const int c = blk * n + c0 + tid;
-        float* rec = p.seg ? p.seg + (size_t(b) * p.max_segments + seg) * 2 * p.W + c : nullptr;
-        float S = p.mode == 0 ? p.state[size_t(slot) * p.W + c] : p.mode == 2 ? rec[0] : 0.f, prod = 1.f;
+        float S = p.mode == 0 ? p.state[size_t(slot) * p.W + c] : 0.f, total = 0.f;
+#pragma unroll 8
         for (int t = 0; t < n_tok; ++t) {
-            const float av = as[t * RF_CH + tid];
-            S = fmaf(av, S, bs[t * RF_CH + tid]);
-            if (p.mode == 1) prod *= av;
-            else as[t * RF_CH + tid] = S;
+            S += fmaf(as[t * RF_CH + tid], S, bs[t * RF_CH + tid]);
+            as[t * RF_CH + tid] = S;
+            total += ls[t * RF_CH + tid];
+            ls[t * RF_CH + tid] = total;
         }
-        if (p.mode == 0) p.state[size_t(slot) * p.W + c] = S;
-        else if (p.mode == 1) { rec[0] = S; rec[p.W] = prod; }
+        if (p.mode == 0) {
+            p.state[size_t(slot) * p.W + c] = S;
+        } else {
+            float* rec = p.seg + (size_t(b) * p.max_segments + seg) * 2 * p.W + c;
+            rec[0] = S;
+            rec[p.W] = total;
+        }
     }
-    if (p.mode == 1) return;
     __syncthreads();
     for (int i = tid; i < n_tok * (RF_CH / 2); i += RF_THREADS) {
         const int tl = i / (RF_CH / 2), ch = 2 * (i % (RF_CH / 2));
         if (ch >= nch) continue;                            // n is even: pairs are whole
         const size_t col = size_t(blk) * n + c0 + ch;
-        const float2 yv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.y + size_t(t0 + tl) * p.ldy + col));
-        *reinterpret_cast<__nv_bfloat162*>(p.out + size_t(t0 + tl) * p.ldo + col) =
-            __floats2bfloat162_rn(as[tl * RF_CH + ch] * gb_gate_act(yv.x, GB_ACT_GELU_TANH), as[tl * RF_CH + ch + 1] * gb_gate_act(yv.y, GB_ACT_GELU_TANH));
+        const float2 S = *reinterpret_cast<const float2*>(as + tl * RF_CH + ch);
+        if (p.mode == 0) {
+            const float2 yv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.y + size_t(t0 + tl) * p.ldy + col));
+            *reinterpret_cast<__nv_bfloat162*>(p.out + size_t(t0 + tl) * p.ldo + col) =
+                __floats2bfloat162_rn(S.x * gb_gate_act(yv.x, GB_ACT_GELU_TANH), S.y * gb_gate_act(yv.y, GB_ACT_GELU_TANH));
+        } else {
+            const float2 l = *reinterpret_cast<const float2*>(ls + tl * RF_CH + ch);
+            float* o = p.local + size_t(t0 + tl) * 2 * p.W + col;
+            *reinterpret_cast<float2*>(o) = S;
+            *reinterpret_cast<float2*>(o + p.W) = make_float2(expf(l.x), expf(l.y));
+        }
     }
+}
+
+// out = (local state + factor * state in front of the token's segment) * gelu_tanh(y), four channels per thread.
+__global__ void __launch_bounds__(128) rglru_finish_kernel(const RfParams p, const int* __restrict__ seq_of) {
+    gb_grid_launch_dependents();
+    gb_grid_wait();
+    const int t = blockIdx.x, c = 4 * (blockIdx.y * 128 + threadIdx.x);
+    const int b = seq_of[t];
+    if (c >= p.W || b < 0 || p.slots[b] < 0) return;
+    const int seg = (t - p.cu[b]) / RF_TOK;
+    const float4 S0 = *reinterpret_cast<const float4*>(p.seg + (size_t(b) * p.max_segments + seg) * 2 * p.W + c);
+    const float* l = p.local + size_t(t) * 2 * p.W + c;
+    const float4 s = *reinterpret_cast<const float4*>(l), f = *reinterpret_cast<const float4*>(l + p.W);
+    const float4 y = gb_load4(p.y, GB_BF16, size_t(t) * p.ldy + c);
+    *reinterpret_cast<uint2*>(p.out + size_t(t) * p.ldo + c) = gb_pack4(make_float4(
+        fmaf(f.x, S0.x, s.x) * gb_gate_act(y.x, GB_ACT_GELU_TANH), fmaf(f.y, S0.y, s.y) * gb_gate_act(y.y, GB_ACT_GELU_TANH),
+        fmaf(f.z, S0.z, s.z) * gb_gate_act(y.z, GB_ACT_GELU_TANH), fmaf(f.w, S0.w, s.w) * gb_gate_act(y.w, GB_ACT_GELU_TANH)));
 }
 
 // ------------------------------------------------------------------------------------------------ single tokens
@@ -287,7 +327,8 @@ __global__ void __launch_bounds__(WARPS * 32) rglru_step_kernel(const RsParams p
         const int c = blk * n + c0 + cl;
         const float log_a = -p.rate[c] * rg_sigmoid(zr + p.b_r[c]);
         float* sp = p.state + size_t(slot) * p.W + c;
-        const float S = fmaf(expf(log_a), *sp, sqrtf(-expm1f(2.f * log_a)) * (rg_sigmoid(zi + p.b_i[c]) * rs_sm[tt * n + c0 + cl]));
+        const float am1 = expm1f(log_a), S0 = *sp;
+        const float S = S0 + fmaf(am1, S0, rg_input(am1, rg_sigmoid(zi + p.b_i[c]) * rs_sm[tt * n + c0 + cl]));
         *sp = S;
         gb_store(p.out, p.out_dtype, size_t(t) * p.ldo + c, S * gb_gate_act(gb_load(p.y, p.dtype, size_t(t) * p.ldy + c), GB_ACT_GELU_TANH));
     }
@@ -338,37 +379,41 @@ GB_API int gb_rglru(const void* u, const void* y, int dtype, long long ldu, cons
 GB_API int gb_rglru_fused_supported(int dtype, int n) { return dtype == GB_BF16 && n > 0 && n % 8 == 0; }
 
 // Prompts, with the gates' products in the same kernels: u, y [T, W] bfloat16; gates [blocks, 2n, n] bfloat16 (n = W / blocks);
-// the rest as gb_rglru.  One launch for steps of at most 64 tokens a sequence, else three.
+// the rest as gb_rglru.  seg: gb_rglru_segment_floats,
+// local: 2 T W floats, both needed where a sequence brings more than 64 tokens.  One launch for steps of at most 64 tokens a sequence, else three.
 GB_API int gb_rglru_fused(const void* u, long long ldu, const void* y, long long ldy, const void* gates, const float* b_r,
                           const float* b_i, const float* rate, float* state, void* out, long long ldo, const int* cu,
-                          const int* slots, const int* qlens, int B, int W, int blocks, int max_qlen, float* seg, cudaStream_t stream) {
+                          const int* slots, const int* qlens, const int* seq_of, int T, int B, int W, int blocks, int max_qlen, float* seg,
+                          float* local, cudaStream_t stream) {
     GB_REQUIRE(W > 0 && blocks > 0 && W % blocks == 0 && gb_rglru_fused_supported(GB_BF16, W / blocks),
                "gb_rglru_fused: %d channels in %d blocks (of a multiple of 8 channels)", W, blocks);
-    GB_REQUIRE(ldu % 8 == 0 && gb_aligned(u, 16) && gb_aligned(gates, 16) && ldy % 2 == 0 && ldo % 2 == 0 && gb_aligned(y, 4) && gb_aligned(out, 4),
+    GB_REQUIRE(ldu % 8 == 0 && gb_aligned(u, 16) && gb_aligned(gates, 16) && ldy % 4 == 0 && ldo % 4 == 0 && gb_aligned(y, 8) && gb_aligned(out, 8) &&
+               gb_aligned(seg, 16) && gb_aligned(local, 16),
                "gb_rglru_fused: misaligned operands");
     if (B == 0 || max_qlen <= 0) return 0;
     RfParams p;
     p.u = (const __nv_bfloat16*)u; p.y = (const __nv_bfloat16*)y; p.gates = (const __nv_bfloat16*)gates; p.b_r = b_r; p.b_i = b_i;
-    p.rate = rate; p.state = state; p.seg = nullptr; p.out = (__nv_bfloat16*)out; p.ldu = ldu; p.ldy = ldy; p.ldo = ldo; p.cu = cu;
+    p.rate = rate; p.state = state; p.seg = nullptr; p.local = nullptr; p.out = (__nv_bfloat16*)out; p.ldu = ldu; p.ldy = ldy; p.ldo = ldo; p.cu = cu;
     p.slots = slots; p.qlens = qlens; p.W = W; p.n = W / blocks; p.slices = (p.n + RF_CH - 1) / RF_CH; p.mode = 0;
     p.max_segments = (max_qlen + RF_TOK - 1) / RF_TOK;
     GB_REQUIRE(B <= 65535 && p.max_segments <= 65535, "gb_rglru_fused: %d sequences of up to %d tokens are too many for one step", B, max_qlen);
     constexpr int SMEM = 2 * (RF_TOK + 2 * RF_CH) * RF_K * 2;
+    static_assert(SMEM >= 3 * RF_TOK * RF_CH * 4 && SMEM <= 48 * 1024, "the walk's arrays lie over the stages");
     const dim3 grid(blocks * p.slices, p.max_segments, B);
     if (p.max_segments == 1) {
         gb_launch(rglru_fused_kernel, grid, dim3(RF_THREADS), SMEM, stream, p);
         GB_LAUNCH_OK("gb_rglru_fused");
         return 0;
     }
-    GB_REQUIRE(seg, "gb_rglru_fused: segments need scratch");
+    GB_REQUIRE(seg && local, "gb_rglru_fused: segments need scratch");
     p.seg = seg;
+    p.local = local;
     p.mode = 1;
     gb_launch(rglru_fused_kernel, grid, dim3(RF_THREADS), SMEM, stream, p);
     GB_LAUNCH_OK("gb_rglru_fused (segments)");
     gb_launch(rglru_carry_kernel, dim3((W + RG_THREADS - 1) / RG_THREADS, B), dim3(RG_THREADS), 0, stream, state, seg, slots, qlens, W, p.max_segments);
     GB_LAUNCH_OK("gb_rglru_fused (carry)");
-    p.mode = 2;
-    gb_launch(rglru_fused_kernel, grid, dim3(RF_THREADS), SMEM, stream, p);
+    gb_launch(rglru_finish_kernel, dim3(T, (W / 4 + 127) / 128), dim3(128), 0, stream, p, seq_of);
     GB_LAUNCH_OK("gb_rglru_fused");
     return 0;
 }

@@ -885,8 +885,10 @@ def rglru_fused(u: torch.Tensor, y: torch.Tensor, gates: torch.Tensor, bias_r: t
     assert gates.shape == (blocks, 2 * n, n) and gates.dtype == u.dtype and gates.is_contiguous()
     need = native.library().gb_rglru_segment_floats(ctx.B, int(ctx.max_qlen), W)
     seg = ctx.ws.get("rglru.segments", (need,), torch.float32) if need else None
+    local = ctx.ws.get("rglru.local", (u.shape[0], 2, W), torch.float32) if need else None
     call("gb_rglru_fused", ptr(u), u.stride(0), ptr(y), y.stride(0), ptr(gates), ptr(bias_r), ptr(bias_i), ptr(rate), ptr(state), ptr(out),
-         out.stride(0), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ctx.B, W, int(blocks), int(ctx.max_qlen), ptr(seg), stream_ptr())
+         out.stride(0), ptr(ctx.cu), ptr(ctx.slots), ptr(ctx.qlens), ptr(ctx.seq_of), u.shape[0], ctx.B, W, int(blocks),
+         int(ctx.max_qlen), ptr(seg), ptr(local), stream_ptr())
     if seg is not None:
         native.count_launches(2)
     return out

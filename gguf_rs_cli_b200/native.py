@@ -186,7 +186,7 @@ _SIGNATURES = {
     "gb_scale_rows": [_P, _P, _I, _I, _P],
     "gb_rglru": [_P, _P, _I, _L, _P, _L, _L, _P, _P, _P, _P, _P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "gb_rglru_fused_supported": [_I, _I],
-    "gb_rglru_fused": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    "gb_rglru_fused": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P],
     "gb_rglru_step": [_P, _P, _I, _L, _L, _P, _I, _P, _P, _P, _P, _P, _I, _L, _P, _P, _I, _I, _I, _P],
     "gb_rglru_segment_floats": [_I, _I, _I],
     "gb_retention": [_P, _P, _P, _I, _L, _P, _P, _I, _I, _F, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P],
