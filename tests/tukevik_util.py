@@ -108,7 +108,7 @@ def make_weights(cfg, seed=0):
     def bias(n, gain=0.3):
         return gain * torch.randn(n, generator=g)
 
-    w["embed"] = torch.randn(V, E, generator=g) * 0.7
+    w["embed"] = torch.randn(V, E, generator=g) * 1.4
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.mix.", layer["mixer"]
         w[f"l{i}.norm1"] = near_one(E)
