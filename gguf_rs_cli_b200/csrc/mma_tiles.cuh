@@ -22,14 +22,30 @@ __device__ __forceinline__ void mma(float (&c)[4], const unsigned (&a)[4], unsig
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// the six products of two numbers of three terms each, smallest first
-__device__ __forceinline__ void mma6(float (&c)[4], const unsigned (&a)[3][4], const unsigned (&b)[3][4], int at) {
-    mma(c, a[0], b[2][at], b[2][at + 1]);
-    mma(c, a[2], b[0][at], b[0][at + 1]);
-    mma(c, a[1], b[1][at], b[1][at + 1]);
-    mma(c, a[0], b[1][at], b[1][at + 1]);
-    mma(c, a[1], b[0][at], b[0][at + 1]);
-    mma(c, a[0], b[0][at], b[0][at + 1]);
+// 16 x 16 of A times 32 columns of B (b and b2: 16 columns each), A and B of three terms: the six products, smallest first,
+// every one of them for all four accumulators before the next, so that an accumulator's products do not follow one
+// another at once
+__device__ __forceinline__ void mma6(float (&c0)[4], float (&c1)[4], float (&c2)[4], float (&c3)[4], const unsigned (&a)[3][4],
+                                     const unsigned (&b)[3][4], const unsigned (&b2)[3][4]) {
+    constexpr int TA[6] = {0, 2, 1, 0, 1, 0}, TB[6] = {2, 0, 1, 1, 0, 0};
+#pragma unroll
+    for (int e = 0; e < 6; ++e) {
+        mma(c0, a[TA[e]], b[TB[e]][0], b[TB[e]][1]);
+        mma(c1, a[TA[e]], b[TB[e]][2], b[TB[e]][3]);
+        mma(c2, a[TA[e]], b2[TB[e]][0], b2[TB[e]][1]);
+        mma(c3, a[TA[e]], b2[TB[e]][2], b2[TB[e]][3]);
+    }
+}
+// the same for a B of one term: three products
+__device__ __forceinline__ void mma3(float (&c0)[4], float (&c1)[4], float (&c2)[4], float (&c3)[4], const unsigned (&a)[3][4],
+                                     const unsigned (&b)[4], const unsigned (&b2)[4]) {
+#pragma unroll
+    for (int e = 2; e >= 0; --e) {
+        mma(c0, a[e], b[0], b[1]);
+        mma(c1, a[e], b[2], b[3]);
+        mma(c2, a[e], b2[0], b2[1]);
+        mma(c3, a[e], b2[2], b2[3]);
+    }
 }
 __device__ __forceinline__ unsigned pack2(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);

@@ -189,14 +189,11 @@ __global__ void __launch_bounds__(2 * N) retention_state_kernel(const RetChunkPa
             for (int e = 0; e < 3; ++e)       // tokens are the inner dimension: a transposed load turns [token][channel]
                 ldsm4_trans(a[e], kp + e * RC_TILE * N + swz<N>(kk * 16 + (lane & 7) + ((lane >> 4) << 3), 2 * warp + ((lane >> 3) & 1)));
 #pragma unroll
-            for (int i2 = 0; i2 < N / 16; ++i2) {
-                unsigned bv[4];
-                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), 2 * i2 + (lane >> 4)));
-#pragma unroll
-                for (int e = 2; e >= 0; --e) {
-                    mma(acc[2 * i2], a[e], bv[0], bv[1]);
-                    mma(acc[2 * i2 + 1], a[e], bv[2], bv[3]);
-                }
+            for (int i4 = 0; i4 < N / 32; ++i4) {
+                unsigned bv[4], bw[4];
+                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + (lane >> 4)));
+                ldsm4_trans(bw, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + 2 + (lane >> 4)));
+                mma3(acc[4 * i4], acc[4 * i4 + 1], acc[4 * i4 + 2], acc[4 * i4 + 3], a, bv, bw);
             }
         }
     }
@@ -287,12 +284,14 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
 #pragma unroll
             for (int e = 0; e < 3; ++e) ldsm4(a[e], qp + e * RC_TILE * N + swz<N>(warp * 16 + (lane & 15), d0 / 8 + 2 * kk + (lane >> 4)));
 #pragma unroll
-            for (int i2 = 0; i2 < N / 16; ++i2) {
-                unsigned bs[3][4];
+            for (int i4 = 0; i4 < N / 32; ++i4) {
+                unsigned bs[3][4], bt[3][4];
 #pragma unroll
-                for (int e = 0; e < 3; ++e) ldsm4_trans(bs[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), 2 * i2 + (lane >> 4)));
-                mma6(acc[2 * i2], a, bs, 0);
-                mma6(acc[2 * i2 + 1], a, bs, 2);
+                for (int e = 0; e < 3; ++e) {
+                    ldsm4_trans(bs[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), 4 * i4 + (lane >> 4)));
+                    ldsm4_trans(bt[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), 4 * i4 + 2 + (lane >> 4)));
+                }
+                mma6(acc[4 * i4], acc[4 * i4 + 1], acc[4 * i4 + 2], acc[4 * i4 + 3], a, bs, bt);
             }
         }
         __syncthreads();
@@ -316,13 +315,15 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
 #pragma unroll
             for (int e = 0; e < 3; ++e) ldsm4(a[e], qp + e * RC_TILE * N + swz<N>(warp * 16 + (lane & 15), 2 * kk + (lane >> 4)));
 #pragma unroll
-            for (int j2 = 0; j2 < RC_TILE / 16; ++j2) {
-                unsigned bk[3][4];
+            for (int j4 = 0; j4 < RC_TILE / 32; ++j4) {
+                unsigned bk[3][4], bl[3][4];
+                const int r = j4 * 32 + (lane & 7) + ((lane >> 4) << 3), c = 2 * kk + ((lane >> 3) & 1);
 #pragma unroll
-                for (int e = 0; e < 3; ++e)
-                    ldsm4(bk[e], kp + e * RC_TILE * N + swz<N>(j2 * 16 + (lane & 7) + ((lane >> 4) << 3), 2 * kk + ((lane >> 3) & 1)));
-                mma6(w[2 * j2], a, bk, 0);
-                mma6(w[2 * j2 + 1], a, bk, 2);
+                for (int e = 0; e < 3; ++e) {
+                    ldsm4(bk[e], kp + e * RC_TILE * N + swz<N>(r, c));
+                    ldsm4(bl[e], kp + e * RC_TILE * N + swz<N>(r + 16, c));
+                }
+                mma6(w[4 * j4], w[4 * j4 + 1], w[4 * j4 + 2], w[4 * j4 + 3], a, bk, bl);
             }
         }
 #pragma unroll
@@ -343,14 +344,11 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
                 split3(w[2 * kk + half][2], w[2 * kk + half][3], a[0][2 * half + 1], a[1][2 * half + 1], a[2][2 * half + 1]);
             }
 #pragma unroll
-            for (int i2 = 0; i2 < N / 16; ++i2) {
-                unsigned bv[4];
-                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), 2 * i2 + (lane >> 4)));
-#pragma unroll
-                for (int e = 2; e >= 0; --e) {
-                    mma(acc[2 * i2], a[e], bv[0], bv[1]);
-                    mma(acc[2 * i2 + 1], a[e], bv[2], bv[3]);
-                }
+            for (int i4 = 0; i4 < N / 32; ++i4) {
+                unsigned bv[4], bw[4];
+                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + (lane >> 4)));
+                ldsm4_trans(bw, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + 2 + (lane >> 4)));
+                mma3(acc[4 * i4], acc[4 * i4 + 1], acc[4 * i4 + 2], acc[4 * i4 + 3], a, bv, bw);
             }
         }
         __syncthreads();

@@ -95,11 +95,21 @@ __global__ void __launch_bounds__(RG_THREADS) rglru_carry_kernel(float* __restri
     if (slot < 0 || n <= 0 || c >= W) return;
     float S = state[size_t(slot) * W + c];
     const int segs = (n + RG_SEGMENT - 1) / RG_SEGMENT;
-    for (int s = 0; s < segs; ++s) {
-        float* rec = seg + (size_t(b) * max_segments + s) * 2 * W + c;
-        const float local = rec[0], am1 = expm1f(rec[W]);
-        rec[0] = S;
-        S += fmaf(am1, S, local);
+    constexpr int AHEAD = 16;                 // segments whose records are on their way together
+    for (int s0 = 0; s0 < segs; s0 += AHEAD) {
+        float* rec = seg + (size_t(b) * max_segments + s0) * 2 * W + c;
+        float local[AHEAD], total[AHEAD];
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            local[j] = s0 + j < segs ? rec[size_t(j) * 2 * W] : 0.f;
+            total[j] = s0 + j < segs ? rec[size_t(j) * 2 * W + W] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; ++j) {
+            if (s0 + j >= segs) break;
+            rec[size_t(j) * 2 * W] = S;
+            S += fmaf(expm1f(total[j]), S, local[j]);
+        }
     }
     state[size_t(slot) * W + c] = S;
 }
