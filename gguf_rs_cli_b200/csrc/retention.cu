@@ -79,89 +79,114 @@ struct RetChunkParams {
     float k_scale, eps, out_scale;
 };
 
+__device__ __forceinline__ void rc_unpack(const uint4& raw, float (&x)[8]) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(h[e]);
+        x[2 * e] = f.x;
+        x[2 * e + 1] = f.y;
+    }
+}
+// eight numbers as three planes of bfloat16 terms, `plane` entries apart
+__device__ __forceinline__ void rc_store_terms(const float (&x)[8], __nv_bfloat16* at, int plane) {
+    using namespace gbmma;
+    uint4 h, m, l;
+    split3(x[0], x[1], h.x, m.x, l.x);
+    split3(x[2], x[3], h.y, m.y, l.y);
+    split3(x[4], x[5], h.z, m.z, l.z);
+    split3(x[6], x[7], h.w, m.w, l.w);
+    *reinterpret_cast<uint4*>(at) = h;
+    *reinterpret_cast<uint4*>(at + plane) = m;
+    *reinterpret_cast<uint4*>(at + 2 * plane) = l;
+}
+
 // 64 rows of q or k: rotated, row r times factor * 2^(row_log2 * (last - r)), as three planes of bfloat16 terms; rows from
-// n on are zero.
-template <int N>
+// n (at least 1) on are zero.  AHEAD pieces of eight entries per thread are on their way together (rows behind the last
+// read the last, so that no load waits for a branch).
+template <int N, int THREADS, int AHEAD>
 __device__ __forceinline__ void rc_load_rotated(const RetChunkParams& p, const __nv_bfloat16* src, int t0, int n, float factor,
                                                 float row_log2, int last, __nv_bfloat16* planes) {
-    using namespace gbmma;
-    constexpr int CH = N / 8;
-    for (int idx = threadIdx.x; idx < RC_TILE * CH; idx += blockDim.x) {
-        const int r = idx / CH, c = idx - r * CH, d = 8 * c;
-        float x[8];
+    constexpr int CH = N / 8, ITEMS = RC_TILE * CH;
+    const bool halves = !p.pairing && p.half > 0 && (p.half & 7) == 0;      // whole pieces are turned with whole pieces
+    for (int base = threadIdx.x; base < ITEMS; base += THREADS * AHEAD) {
+        uint4 own[AHEAD], oth[AHEAD];
+        float4 ang[AHEAD][4];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = 0.f;
-        if (r < n) {
+        for (int u = 0; u < AHEAD; ++u) {
+            const int idx = min(base + u * THREADS, ITEMS - 1), r = min(idx / CH, n - 1), d = 8 * (idx % CH);
             const __nv_bfloat16* row = src + size_t(t0 + r) * p.ld;
-            const uint4 own = *reinterpret_cast<const uint4*>(row + d);
-            const __nv_bfloat162* o2 = reinterpret_cast<const __nv_bfloat162*>(&own);
+            own[u] = __ldg(reinterpret_cast<const uint4*>(row + d));
+            if (halves) {
+                const bool turned = d < 2 * p.half, first = d < p.half;
+                oth[u] = __ldg(reinterpret_cast<const uint4*>(row + (!turned ? d : first ? d + p.half : d - p.half)));
+                const float4* a = reinterpret_cast<const float4*>(p.angles + size_t(t0 + r) * p.half + (!turned ? 0 : first ? d : d - p.half));
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float2 f = __bfloat1622float2(o2[e]);
-                x[2 * e] = f.x;
-                x[2 * e + 1] = f.y;
+                for (int e = 0; e < 4; ++e) ang[u][e] = __ldg(a + e);
             }
-            const float2* ang = p.angles + size_t(t0 + r) * p.half;
-            if (d < 2 * p.half) {
-                if (!p.pairing && (p.half & 7) == 0) {
+        }
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u) {
+            const int idx = base + u * THREADS;
+            if (idx >= ITEMS) break;
+            const int r = idx / CH, c = idx - r * CH, d = 8 * c;
+            float x[8];
+            rc_unpack(own[u], x);
+            if (halves) {
+                if (d < 2 * p.half) {
                     const bool first = d < p.half;
-                    const int i0 = first ? d : d - p.half;
-                    const uint4 oth = *reinterpret_cast<const uint4*>(row + (first ? d + p.half : d - p.half));
-                    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&oth);
+                    float o[8];
+                    rc_unpack(oth[u], o);
 #pragma unroll
                     for (int e = 0; e < 8; ++e) {
-                        const float2 f = __bfloat1622float2(h2[e >> 1]), cs = ang[i0 + e];
-                        const float other = (e & 1) ? f.y : f.x;
+                        const float4 a = ang[u][e >> 1];
+                        const float cs = (e & 1) ? a.z : a.x, sn = (e & 1) ? a.w : a.y;
+                        float y0, y1;
+                        gb_rotate(first ? x[e] : o[e], first ? o[e] : x[e], cs, sn, y0, y1);
+                        x[e] = first ? y0 : y1;
+                    }
+                }
+            } else if (r < n) {
+                const __nv_bfloat16* row = src + size_t(t0 + r) * p.ld;
+                const float2* a = p.angles + size_t(t0 + r) * p.half;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const int dd = d + e;
+                    if (dd < 2 * p.half) {
+                        const bool first = p.pairing ? (dd & 1) == 0 : dd < p.half;
+                        const float2 cs = a[p.pairing ? dd >> 1 : first ? dd : dd - p.half];
+                        const float other = __bfloat162float(row[p.pairing ? dd ^ 1 : first ? dd + p.half : dd - p.half]);
                         float y0, y1;
                         gb_rotate(first ? x[e] : other, first ? other : x[e], cs.x, cs.y, y0, y1);
                         x[e] = first ? y0 : y1;
                     }
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) {
-                        const int dd = d + e;
-                        if (dd < 2 * p.half) {
-                            const bool first = p.pairing ? (dd & 1) == 0 : dd < p.half;
-                            const int i = p.pairing ? dd >> 1 : first ? dd : dd - p.half;
-                            const float other = __bfloat162float(row[p.pairing ? dd ^ 1 : first ? dd + p.half : dd - p.half]);
-                            const float2 cs = ang[i];
-                            float y0, y1;
-                            gb_rotate(first ? x[e] : other, first ? other : x[e], cs.x, cs.y, y0, y1);
-                            x[e] = first ? y0 : y1;
-                        }
-                    }
                 }
             }
-            const float f = row_log2 != 0.f ? factor * exp2f(row_log2 * float(last - r)) : factor;
+            const float f = r >= n ? 0.f : row_log2 != 0.f ? factor * exp2f(row_log2 * float(last - r)) : factor;
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] *= f;
+            for (int e = 0; e < 8; ++e) x[e] = r < n ? x[e] * f : 0.f;
+            rc_store_terms(x, planes + gbmma::swz<N>(r, c), RC_TILE * N);
         }
-        uint4 h, m, l;
-        split3(x[0], x[1], h.x, m.x, l.x);
-        split3(x[2], x[3], h.y, m.y, l.y);
-        split3(x[4], x[5], h.z, m.z, l.z);
-        split3(x[6], x[7], h.w, m.w, l.w);
-        const int at = swz<N>(r, c);
-        *reinterpret_cast<uint4*>(planes + at) = h;
-        *reinterpret_cast<uint4*>(planes + RC_TILE * N + at) = m;
-        *reinterpret_cast<uint4*>(planes + 2 * RC_TILE * N + at) = l;
     }
 }
 
-template <int N>
+template <int N, int THREADS>
 __device__ __forceinline__ void rc_load_values(const RetChunkParams& p, const __nv_bfloat16* src, int t0, int n, __nv_bfloat16* vt) {
-    constexpr int CH = N / 8;
-    for (int idx = threadIdx.x; idx < RC_TILE * CH; idx += blockDim.x) {
+    constexpr int CH = N / 8, ITEMS = RC_TILE * CH;
+#pragma unroll
+    for (int base = 0; base < ITEMS; base += THREADS) {
+        const int idx = base + threadIdx.x;
+        if (ITEMS % THREADS && idx >= ITEMS) break;
         const int r = idx / CH, c = idx - r * CH;
-        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-        if (r < n) raw = *reinterpret_cast<const uint4*>(src + size_t(t0 + r) * p.ld + 8 * c);
+        uint4 raw = __ldg(reinterpret_cast<const uint4*>(src + size_t(t0 + min(r, n - 1)) * p.ld + 8 * c));
+        if (r >= n) raw = make_uint4(0u, 0u, 0u, 0u);
         *reinterpret_cast<uint4*>(vt + gbmma::swz<N>(r, c)) = raw;
     }
 }
 
 // seg[b * n_seg + s, h] = sum_j g^(n-1-j) k'_j v_j^T over the segment's n tokens.  N / 16 warps, 16 key channels each.
 template <int N>
-__global__ void __launch_bounds__(2 * N) retention_state_kernel(const RetChunkParams p) {
+__global__ void __launch_bounds__(2 * N, 2) retention_state_kernel(const RetChunkParams p) {
     using namespace gbmma;
     extern __shared__ __align__(128) unsigned char rc_smem[];
     __nv_bfloat16* kp = reinterpret_cast<__nv_bfloat16*>(rc_smem);          // [3][64][N]
@@ -179,8 +204,8 @@ __global__ void __launch_bounds__(2 * N) retention_state_kernel(const RetChunkPa
     for (int j0 = 0; j0 < n; j0 += RC_TILE) {
         const int nb = min(RC_TILE, n - j0);
         __syncthreads();
-        rc_load_rotated<N>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, lg, n - 1 - j0, kp);
-        rc_load_values<N>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
+        rc_load_rotated<N, 2 * N, 2>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, lg, n - 1 - j0, kp);
+        rc_load_values<N, 2 * N>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
         __syncthreads();
 #pragma unroll
         for (int kk = 0; kk < RC_TILE / 16; ++kk) {
@@ -256,27 +281,32 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
     const int t0 = p.cu[b] + s * RC_SEG, rows = min(RC_TILE, n - q0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float lg = p.log2_decay[h];
-    rc_load_rotated<N>(p, p.q + size_t(h) * N, t0 + q0, rows, 1.f, 0.f, 0, qp);
+    rc_load_rotated<N, 128, 4>(p, p.q + size_t(h) * N, t0 + q0, rows, 1.f, 0.f, 0, qp);
     float acc[N / 8][4];
 #pragma unroll
     for (int i = 0; i < N / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    // ---- q' S0, 32 rows of S0 at a time
+    // ---- q' S0, 32 rows of S0 at a time, the next rows on their way meanwhile
     const float* S0 = p.seg + (size_t(unit) * p.H + h) * size_t(N) * N;
-    for (int d0 = 0; d0 < N; d0 += 32) {
-        for (int idx = threadIdx.x; idx < 32 * (N / 8); idx += 128) {
-            const int r = idx / (N / 8), c = idx - r * (N / 8);
+    constexpr int PIECES = 32 * (N / 8) / 128;                              // pieces of eight entries per thread
+    float4 next[PIECES][2];
+    auto fetch = [&](int d0) {
+#pragma unroll
+        for (int u = 0; u < PIECES; ++u) {
+            const int idx = u * 128 + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
             const float4* src = reinterpret_cast<const float4*>(S0 + size_t(d0 + r) * N + 8 * c);
-            const float4 x = src[0], y = src[1];
-            uint4 hh, m, l;
-            split3(x.x, x.y, hh.x, m.x, l.x);
-            split3(x.z, x.w, hh.y, m.y, l.y);
-            split3(y.x, y.y, hh.z, m.z, l.z);
-            split3(y.z, y.w, hh.w, m.w, l.w);
-            const int at = swz<N>(r, c);
-            *reinterpret_cast<uint4*>(kp + at) = hh;
-            *reinterpret_cast<uint4*>(kp + 32 * N + at) = m;
-            *reinterpret_cast<uint4*>(kp + 64 * N + at) = l;
+            next[u][0] = __ldg(src);
+            next[u][1] = __ldg(src + 1);
         }
+    };
+    fetch(0);
+    for (int d0 = 0; d0 < N; d0 += 32) {
+#pragma unroll
+        for (int u = 0; u < PIECES; ++u) {
+            const int idx = u * 128 + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
+            const float x[8] = {next[u][0].x, next[u][0].y, next[u][0].z, next[u][0].w, next[u][1].x, next[u][1].y, next[u][1].z, next[u][1].w};
+            rc_store_terms(x, kp + swz<N>(r, c), 32 * N);
+        }
+        if (d0 + 32 < N) fetch(d0 + 32);
         __syncthreads();
 #pragma unroll
         for (int kk = 0; kk < 2; ++kk) {
@@ -303,8 +333,8 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
     // ---- the segment's own keys up to each query
     for (int j0 = 0; j0 <= q0; j0 += RC_TILE) {
         const int nb = min(RC_TILE, n - j0);
-        rc_load_rotated<N>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, 0.f, 0, kp);
-        rc_load_values<N>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
+        rc_load_rotated<N, 128, 4>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, 0.f, 0, kp);
+        rc_load_values<N, 128>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
         __syncthreads();
         float w[RC_TILE / 8][4];
 #pragma unroll
