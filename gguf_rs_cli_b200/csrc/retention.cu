@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(2 * N, 2) retention_state_kernel(const RetChun
     for (int j0 = 0; j0 < n; j0 += RC_TILE) {
         const int nb = min(RC_TILE, n - j0);
         __syncthreads();
-        rc_load_rotated<N, 2 * N, 2>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, lg, n - 1 - j0, kp);
+        rc_load_rotated<N, 2 * N, 1>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, lg, n - 1 - j0, kp);
         rc_load_values<N, 2 * N>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
         __syncthreads();
 #pragma unroll
@@ -262,47 +262,55 @@ __global__ void __launch_bounds__(128) retention_carry_kernel(float4* __restrict
     *sp = S;
 }
 
-// 64 queries of one head: four warps of 16, all N value columns each.
+// 64 queries of one head.  A warp has 16 of them and, where the head's size is a multiple of 64, half of the value columns
+// (two warps share their queries): it then makes the scores of half of the keys, and the weights go through shared memory.
+template <int N> struct RcOut {
+    static constexpr int HALVES = N % 64 == 0 ? 2 : 1, THREADS = 128 * HALVES, COLS = N / HALVES, KEYS = RC_TILE / HALVES;
+};
+
 template <int N>
-__global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams p) {
+__global__ void __launch_bounds__(RcOut<N>::THREADS, 2) retention_out_kernel(const RetChunkParams p) {
     using namespace gbmma;
+    using L = RcOut<N>;
     extern __shared__ __align__(128) unsigned char rc_smem[];
+    __shared__ float ss_part[L::HALVES][RC_TILE];
     __nv_bfloat16* qp = reinterpret_cast<__nv_bfloat16*>(rc_smem);          // [3][64][N]
-    __nv_bfloat16* kp = qp + 3 * RC_TILE * N;                               // [3][64][N], before that slices of S
-    __nv_bfloat16* vt = kp + 3 * RC_TILE * N;                               // [64][N]
+    __nv_bfloat16* kp = qp + 3 * RC_TILE * N;                               // slices of S; then keys [3][64][N]
+    __nv_bfloat16* vt = kp + 3 * RC_TILE * (N > RC_TILE ? N : RC_TILE);     // [64][N]
+    __nv_bfloat16* wp = kp;                                                 // weights [3][64][64], over the keys when those are used up
     gb_grid_launch_dependents();
     gb_grid_wait();
     constexpr int TILES = RC_SEG / RC_TILE;
-    const int unit = blockIdx.x / TILES, tile = blockIdx.x % TILES, h = blockIdx.y;
+    const int unit = blockIdx.x / TILES, tile = TILES - 1 - blockIdx.x % TILES, h = blockIdx.y;
     const int b = unit / p.n_seg, s = unit % p.n_seg;
     const int n = min(RC_SEG, p.qlens[b] - s * RC_SEG);                     // tokens of the segment
     const int q0 = tile * RC_TILE;
     if (p.slots[b] < 0 || q0 >= n) return;
     const int t0 = p.cu[b] + s * RC_SEG, rows = min(RC_TILE, n - q0);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = (threadIdx.x >> 5) & 3, half = threadIdx.x >> 7, lane = threadIdx.x & 31, col0 = half * L::COLS;
     const float lg = p.log2_decay[h];
-    rc_load_rotated<N, 128, 4>(p, p.q + size_t(h) * N, t0 + q0, rows, 1.f, 0.f, 0, qp);
-    float acc[N / 8][4];
-#pragma unroll
-    for (int i = 0; i < N / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     // ---- q' S0, 32 rows of S0 at a time, the next rows on their way meanwhile
     const float* S0 = p.seg + (size_t(unit) * p.H + h) * size_t(N) * N;
-    constexpr int PIECES = 32 * (N / 8) / 128;                              // pieces of eight entries per thread
+    constexpr int PIECES = 32 * (N / 8) / L::THREADS;                       // pieces of eight entries per thread
     float4 next[PIECES][2];
     auto fetch = [&](int d0) {
 #pragma unroll
         for (int u = 0; u < PIECES; ++u) {
-            const int idx = u * 128 + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
+            const int idx = u * L::THREADS + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
             const float4* src = reinterpret_cast<const float4*>(S0 + size_t(d0 + r) * N + 8 * c);
             next[u][0] = __ldg(src);
             next[u][1] = __ldg(src + 1);
         }
     };
     fetch(0);
+    rc_load_rotated<N, L::THREADS, 2>(p, p.q + size_t(h) * N, t0 + q0, rows, 1.f, 0.f, 0, qp);
+    float acc[L::COLS / 8][4];
+#pragma unroll
+    for (int i = 0; i < L::COLS / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     for (int d0 = 0; d0 < N; d0 += 32) {
 #pragma unroll
         for (int u = 0; u < PIECES; ++u) {
-            const int idx = u * 128 + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
+            const int idx = u * L::THREADS + threadIdx.x, r = idx / (N / 8), c = idx - r * (N / 8);
             const float x[8] = {next[u][0].x, next[u][0].y, next[u][0].z, next[u][0].w, next[u][1].x, next[u][1].y, next[u][1].z, next[u][1].w};
             rc_store_terms(x, kp + swz<N>(r, c), 32 * N);
         }
@@ -314,40 +322,41 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
 #pragma unroll
             for (int e = 0; e < 3; ++e) ldsm4(a[e], qp + e * RC_TILE * N + swz<N>(warp * 16 + (lane & 15), d0 / 8 + 2 * kk + (lane >> 4)));
 #pragma unroll
-            for (int i4 = 0; i4 < N / 32; ++i4) {
+            for (int i4 = 0; i4 < L::COLS / 32; ++i4) {
                 unsigned bs[3][4], bt[3][4];
+                const int c = col0 / 8 + 4 * i4 + (lane >> 4);
 #pragma unroll
                 for (int e = 0; e < 3; ++e) {
-                    ldsm4_trans(bs[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), 4 * i4 + (lane >> 4)));
-                    ldsm4_trans(bt[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), 4 * i4 + 2 + (lane >> 4)));
+                    ldsm4_trans(bs[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), c));
+                    ldsm4_trans(bt[e], kp + e * 32 * N + swz<N>(kk * 16 + (lane & 15), c + 2));
                 }
                 mma6(acc[4 * i4], acc[4 * i4 + 1], acc[4 * i4 + 2], acc[4 * i4 + 3], a, bs, bt);
             }
         }
         __syncthreads();
     }
-    const int i0 = q0 + warp * 16 + (lane >> 2), i1 = i0 + 8;               // this thread's two queries within the segment
+    const int r0 = warp * 16 + (lane >> 2), i0 = q0 + r0, i1 = i0 + 8;      // this thread's two queries: in the tile, in the segment
     const float g0 = exp2f(lg * float(i0 + 1)), g1 = exp2f(lg * float(i1 + 1));
 #pragma unroll
-    for (int i = 0; i < N / 8; ++i) { acc[i][0] *= g0; acc[i][1] *= g0; acc[i][2] *= g1; acc[i][3] *= g1; }
+    for (int i = 0; i < L::COLS / 8; ++i) { acc[i][0] *= g0; acc[i][1] *= g0; acc[i][2] *= g1; acc[i][3] *= g1; }
     // ---- the segment's own keys up to each query
     for (int j0 = 0; j0 <= q0; j0 += RC_TILE) {
         const int nb = min(RC_TILE, n - j0);
-        rc_load_rotated<N, 128, 4>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, 0.f, 0, kp);
-        rc_load_values<N, 128>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
+        rc_load_rotated<N, L::THREADS, 2>(p, p.k + size_t(h) * N, t0 + j0, nb, p.k_scale, 0.f, 0, kp);
+        rc_load_values<N, L::THREADS>(p, p.v + size_t(h) * N, t0 + j0, nb, vt);
         __syncthreads();
-        float w[RC_TILE / 8][4];
+        float w[L::KEYS / 8][4];
 #pragma unroll
-        for (int j = 0; j < RC_TILE / 8; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
+        for (int j = 0; j < L::KEYS / 8; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
 #pragma unroll 2
         for (int kk = 0; kk < N / 16; ++kk) {
             unsigned a[3][4];
 #pragma unroll
             for (int e = 0; e < 3; ++e) ldsm4(a[e], qp + e * RC_TILE * N + swz<N>(warp * 16 + (lane & 15), 2 * kk + (lane >> 4)));
 #pragma unroll
-            for (int j4 = 0; j4 < RC_TILE / 32; ++j4) {
+            for (int j4 = 0; j4 < L::KEYS / 32; ++j4) {
                 unsigned bk[3][4], bl[3][4];
-                const int r = j4 * 32 + (lane & 7) + ((lane >> 4) << 3), c = 2 * kk + ((lane >> 3) & 1);
+                const int r = half * L::KEYS + j4 * 32 + (lane & 7) + ((lane >> 4) << 3), c = 2 * kk + ((lane >> 3) & 1);
 #pragma unroll
                 for (int e = 0; e < 3; ++e) {
                     ldsm4(bk[e], kp + e * RC_TILE * N + swz<N>(r, c));
@@ -356,28 +365,37 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
                 mma6(w[4 * j4], w[4 * j4 + 1], w[4 * j4 + 2], w[4 * j4 + 3], a, bk, bl);
             }
         }
+        __syncthreads();                                                    // the keys are used up
 #pragma unroll
-        for (int j = 0; j < RC_TILE / 8; ++j) {
-            const int ja = j0 + 8 * j + 2 * (lane & 3);
+        for (int j = 0; j < L::KEYS / 8; ++j) {
+            const int jl = half * L::KEYS + 8 * j + 2 * (lane & 3), ja = j0 + jl;
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int dist = (e < 2 ? i0 : i1) - ja - (e & 1);
                 w[j][e] = dist >= 0 ? w[j][e] * exp2f(lg * float(dist)) : 0.f;
             }
+#pragma unroll
+            for (int rr = 0; rr < 2; ++rr) {
+                unsigned th, tm, tl;
+                split3(w[j][2 * rr], w[j][2 * rr + 1], th, tm, tl);
+                __nv_bfloat16* at = wp + swz<RC_TILE>(r0 + 8 * rr, jl >> 3) + (jl & 7);
+                *reinterpret_cast<unsigned*>(at) = th;
+                *reinterpret_cast<unsigned*>(at + RC_TILE * RC_TILE) = tm;
+                *reinterpret_cast<unsigned*>(at + 2 * RC_TILE * RC_TILE) = tl;
+            }
         }
+        __syncthreads();
 #pragma unroll
         for (int kk = 0; kk < RC_TILE / 16; ++kk) {
             unsigned a[3][4];
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                split3(w[2 * kk + half][0], w[2 * kk + half][1], a[0][2 * half], a[1][2 * half], a[2][2 * half]);
-                split3(w[2 * kk + half][2], w[2 * kk + half][3], a[0][2 * half + 1], a[1][2 * half + 1], a[2][2 * half + 1]);
-            }
+            for (int e = 0; e < 3; ++e) ldsm4(a[e], wp + e * RC_TILE * RC_TILE + swz<RC_TILE>(warp * 16 + (lane & 15), 2 * kk + (lane >> 4)));
 #pragma unroll
-            for (int i4 = 0; i4 < N / 32; ++i4) {
+            for (int i4 = 0; i4 < L::COLS / 32; ++i4) {
                 unsigned bv[4], bw[4];
-                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + (lane >> 4)));
-                ldsm4_trans(bw, vt + swz<N>(kk * 16 + (lane & 15), 4 * i4 + 2 + (lane >> 4)));
+                const int c = col0 / 8 + 4 * i4 + (lane >> 4);
+                ldsm4_trans(bv, vt + swz<N>(kk * 16 + (lane & 15), c));
+                ldsm4_trans(bw, vt + swz<N>(kk * 16 + (lane & 15), c + 2));
                 mma3(acc[4 * i4], acc[4 * i4 + 1], acc[4 * i4 + 2], acc[4 * i4 + 3], a, bv, bw);
             }
         }
@@ -386,26 +404,32 @@ __global__ void __launch_bounds__(128) retention_out_kernel(const RetChunkParams
     // ---- unit root mean square per row, gate, factor
     float ss0 = 0.f, ss1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < N / 8; ++i) {
+    for (int i = 0; i < L::COLS / 8; ++i) {
         ss0 = fmaf(acc[i][0], acc[i][0], ss0); ss0 = fmaf(acc[i][1], acc[i][1], ss0);
         ss1 = fmaf(acc[i][2], acc[i][2], ss1); ss1 = fmaf(acc[i][3], acc[i][3], ss1);
     }
 #pragma unroll
     for (int o = 1; o < 4; o <<= 1) { ss0 += __shfl_xor_sync(0xffffffffu, ss0, o); ss1 += __shfl_xor_sync(0xffffffffu, ss1, o); }
+    if (L::HALVES > 1) {
+        if ((lane & 3) == 0) { ss_part[half][r0] = ss0; ss_part[half][r0 + 8] = ss1; }
+        __syncthreads();
+        ss0 = ss_part[0][r0] + ss_part[L::HALVES - 1][r0];
+        ss1 = ss_part[0][r0 + 8] + ss_part[L::HALVES - 1][r0 + 8];
+    }
     const float f0 = p.out_scale / sqrtf(ss0 / float(N) + p.eps), f1 = p.out_scale / sqrtf(ss1 / float(N) + p.eps);
-    const size_t col = size_t(h) * N + 2 * (lane & 3);
+    const size_t col = size_t(h) * N + col0 + 2 * (lane & 3);
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int r = half ? i1 : i0;
+    for (int rr = 0; rr < 2; ++rr) {
+        const int r = rr ? i1 : i0;
         if (r >= n) continue;
         const __nv_bfloat16* gr = p.gate + size_t(t0 + r) * p.ldg + col;
         __nv_bfloat16* orow = p.out + size_t(t0 + r) * p.ldo + col;
-        const float f = half ? f1 : f0;
+        const float f = rr ? f1 : f0;
 #pragma unroll
-        for (int i = 0; i < N / 8; ++i) {
+        for (int i = 0; i < L::COLS / 8; ++i) {
             const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + 8 * i));
             *reinterpret_cast<__nv_bfloat162*>(orow + 8 * i) =
-                __floats2bfloat162_rn(acc[i][2 * half] * f * (z.x / (1.f + expf(-z.x))), acc[i][2 * half + 1] * f * (z.y / (1.f + expf(-z.y))));
+                __floats2bfloat162_rn(acc[i][2 * rr] * f * (z.x / (1.f + expf(-z.x))), acc[i][2 * rr + 1] * f * (z.y / (1.f + expf(-z.y))));
         }
     }
 }
@@ -577,7 +601,7 @@ GB_API long long gb_retention_chunk_floats(int B, int max_qlen, int H, int D, in
 }
 
 template <int N> static int retention_chunks_launch(const RetChunkParams& p, int B, cudaStream_t stream) {
-    constexpr int SMEM_STATE = (3 * RC_TILE * N + RC_TILE * N) * 2, SMEM_OUT = (6 * RC_TILE * N + RC_TILE * N) * 2;
+    constexpr int SMEM_STATE = (3 * RC_TILE * N + RC_TILE * N) * 2, SMEM_OUT = (4 * RC_TILE * N + 3 * RC_TILE * (N > RC_TILE ? N : RC_TILE)) * 2;
     static bool configured = false;
     if (!configured) {
         if (cudaFuncSetAttribute(retention_state_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE) != cudaSuccess ||
@@ -591,7 +615,7 @@ template <int N> static int retention_chunks_launch(const RetChunkParams& p, int
     gb_launch(retention_carry_kernel, dim3(B, p.H, (E4 + 127) / 128), dim3(128), 0, stream, (float4*)p.state, (float4*)p.seg, p.log2_decay,
               p.slots, p.qlens, p.H, E4, p.n_seg);
     GB_LAUNCH_OK("gb_retention_chunks (carry)");
-    gb_launch(retention_out_kernel<N>, dim3(B * p.n_seg * (RC_SEG / RC_TILE), p.H), dim3(128), SMEM_OUT, stream, p);
+    gb_launch(retention_out_kernel<N>, dim3(B * p.n_seg * (RC_SEG / RC_TILE), p.H), dim3(RcOut<N>::THREADS), SMEM_OUT, stream, p);
     GB_LAUNCH_OK("gb_retention_chunks");
     return 0;
 }
