@@ -157,7 +157,8 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
     // with a softcap or a distance bias the scores are brought into the exponent's units before the softmax
     const bool capped = EXACT && p.softcap > 0.f, biased = EXACT && (p.slopes || capped);
     const float slope2 = EXACT && p.slopes ? p.slopes[h] * 1.4426950408889634f : 0.f;
-    const float to_cap = capped ? p.scale_log2 / (p.softcap * 1.4426950408889634f) : 0.f, cap2 = p.softcap * 1.4426950408889634f;
+    // c tanh(x) = c - 2c / (1 + e^(2x)): an error of a few units in the last place of the cap, as the rounding of c tanh(x) has
+    const float cap2 = p.softcap * 1.4426950408889634f, to_cap = capped ? 2.f * p.scale_log2 / p.softcap : 0.f;
     const float sl2 = biased ? 1.f : p.scale_log2;
 
     float o[OT][4];
@@ -204,7 +205,7 @@ __global__ void __launch_bounds__(AP_THREADS, EXACT ? 1 : 2) attention_prefill_k
             if (biased) {
                 const float d0 = float(pq0 - key0 - 8 * j), d1 = float(pq1 - key0 - 8 * j);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[j][e] = capped ? cap2 * tanhf(s[j][e] * to_cap) : s[j][e] * p.scale_log2;
+                for (int e = 0; e < 4; ++e) s[j][e] = capped ? cap2 - __fdividef(2.f * cap2, 1.f + exp2f(s[j][e] * to_cap)) : s[j][e] * p.scale_log2;
                 s[j][0] -= slope2 * d0; s[j][1] -= slope2 * (d0 - 1.f);
                 s[j][2] -= slope2 * d1; s[j][3] -= slope2 * (d1 - 1.f);
             }
